@@ -5,4 +5,5 @@ from .pafevik import PafevikConfig
 from .zalunex import ZalunexConfig
 from .pogezen import PogezenConfig
 from .figudra import FigudraConfig
+from .vesidra import VesidraConfig
 from .registry import AutoConfig, Architecture, lookup, lookup_config, register_architecture, registered

@@ -1,6 +1,6 @@
 // Prompt attention on the fifth-generation tensor cores (tcgen05) with the accumulators in tensor
-// memory, for head sizes 64 and 128, bfloat16, causal, with or without per-head score slopes (ALiBi),
-// over the paged cache. The description below
+// memory, for head sizes 64 and 128 (and keys of 192 entries beside values of 128), bfloat16, causal, with or
+// without per-head score slopes (ALiBi), over the paged cache. The description below
 // is for head size 64; with 128 the tiles of Q, K and V are two blocks of 64 dims, S takes two groups
 // of matrix instructions, O two (one per 64 dims of the output), and one block fits on an SM.
 //
@@ -99,10 +99,14 @@ constexpr int SOFTMAX_THREADS = TQ;                 // one thread per query row
 // tensor memory accelerator for the pages
 constexpr int BLOCK_THREADS = SOFTMAX_THREADS + 64;
 
+// DK, DV: entries of a query or key row and of a value row (64 or 128 alike, or 192 beside 128).
 // BIAS: a per-head slope times the key's position is added to the raw scores, formed in bfloat16 as
 // the reference forms it.
-template <int D, bool BIAS>
-__global__ void __launch_bounds__(BLOCK_THREADS, D == 64 ? 2 : 1)
+// WIDE: the softmax weights meet V as two bfloat16 terms (the rounded weight, then what the rounding left: 16
+// bits of mantissa). The terms of a page, 32 columns each, together take the place of its S; O += P V is two
+// groups of matrix instructions on the same V tile.
+template <int DK, int DV, bool BIAS, bool WIDE>
+__global__ void __launch_bounds__(BLOCK_THREADS, DK == 64 ? 2 : 1)
 attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k_pool,
                     const __nv_bfloat16* __restrict__ v_pool, __nv_bfloat16* __restrict__ out, StepBatch sb,
                     const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, TcParams p,
@@ -111,21 +115,22 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   extern __shared__ unsigned char smem_dyn[];
   // 1024-byte alignment: the swizzle pattern is a function of address bits 4..9
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(smem_dyn) + 1023) & ~uintptr_t(1023));
-  constexpr int TILE_Q_BYTES = TQ * D * 2;       // 16 or 32 KB
-  constexpr int TILE_KV_BYTES = KEYS * D * 2;    // 8 or 16 KB
-  // tensor memory: three S buffers of 64 columns (page i uses buffer i % 3), O at [192, 192 + D). P of a
+  constexpr int TILE_Q_BYTES = TQ * DK * 2;      // 16, 32 or 48 KB
+  constexpr int TILE_K_BYTES = KEYS * DK * 2;    // 8, 16 or 24 KB
+  constexpr int TILE_V_BYTES = KEYS * DV * 2;    // 8 or 16 KB
+  // tensor memory: three S buffers of 64 columns (page i uses buffer i % 3), O at [192, 192 + DV). P of a
   // page (64 keys as bfloat16 pairs, 32 columns) takes the place of its S: a thread has its row of S in
   // registers before it writes its row of P, nobody else touches that row, and the S of three pages later
   // is issued after the O += P V that reads this P (the tensor pipe runs in order). With three buffers S
   // runs two pages ahead of the softmax, so the softmax does not wait for a matrix product that was
   // issued only when the slowest warp finished the page before.
-  constexpr uint32_t TMEM_O = 192, TMEM_COLS = (D == 64) ? 256 : 512;
+  constexpr uint32_t TMEM_O = 192, TMEM_COLS = (DV == 64) ? 256 : 512;
   unsigned char* q_tile = smem;
   unsigned char* k_ring = q_tile + TILE_Q_BYTES;                      // STAGES_TC pages
-  unsigned char* v_ring = k_ring + STAGES_TC * TILE_KV_BYTES;         // STAGES_TC pages
+  unsigned char* v_ring = k_ring + STAGES_TC * TILE_K_BYTES;          // STAGES_TC pages
   // barriers: [0..2] S buffer written; [3..6] O updated (page % 4); [7..9] P written (page % 3);
   // then per stage: page landed, stage free again
-  uint64_t* bars = reinterpret_cast<uint64_t*>(v_ring + STAGES_TC * TILE_KV_BYTES);
+  uint64_t* bars = reinterpret_cast<uint64_t*>(v_ring + STAGES_TC * TILE_V_BYTES);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 10 + 2 * STAGES_TC);
 
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
@@ -161,17 +166,18 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   // The copy warp's first lane sets the barriers up and asks for the first pages at once (their numbers
   // read by the warp's lanes, one each): they are on their way while the other warps fetch Q and tensor
   // memory is allocated. Nobody else touches a barrier before the block-wide barrier below.
-  constexpr uint32_t PAGE_BYTES = 2 * TILE_KV_BYTES;
+  constexpr uint32_t PAGE_BYTES = TILE_K_BYTES + TILE_V_BYTES;
   auto ask_page = [&](int b, int page) {
     const int st = b % STAGES_TC;
     const int y = (page * p.kv_heads + g) * KEYS;   // first row of the page in the pool seen as [rows][D]
     const uint32_t full = bar_k + 8 * st;
     mbar_expect_tx(full, PAGE_BYTES);
 #pragma unroll
-    for (int blk = 0; blk < D / 64; ++blk) {
-      tma_load_2d(smem_u32(k_ring + st * TILE_KV_BYTES + blk * (KEYS * 128)), &k_map, blk * 64, y, full);
-      tma_load_2d(smem_u32(v_ring + st * TILE_KV_BYTES + blk * (KEYS * 128)), &v_map, blk * 64, y, full);
-    }
+    for (int blk = 0; blk < DK / 64; ++blk)
+      tma_load_2d(smem_u32(k_ring + st * TILE_K_BYTES + blk * (KEYS * 128)), &k_map, blk * 64, y, full);
+#pragma unroll
+    for (int blk = 0; blk < DV / 64; ++blk)
+      tma_load_2d(smem_u32(v_ring + st * TILE_V_BYTES + blk * (KEYS * 128)), &v_map, blk * 64, y, full);
   };
   int first_pages = 0;   // the copy warp's lanes: the number of page b = lane
   if (copy_warp) {
@@ -200,10 +206,10 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
   if (!mma_warp && !copy_warp) {
     // Q tile: rows of the tile, zero beyond the valid tokens
     const uint32_t qs = smem_u32(q_tile);
-    for (int i = tid; i < TQ * (D / 8); i += SOFTMAX_THREADS) {
-      const int r = i / (D / 8), c = i % (D / 8);
+    for (int i = tid; i < TQ * (DK / 8); i += SOFTMAX_THREADS) {
+      const int r = i / (DK / 8), c = i % (DK / 8);
       if (r < tok_valid)
-        cp_async16(qs + swz_tc<TQ>(r, c), q + (size_t(start + q0 + r) * p.heads + h) * D + c * 8);
+        cp_async16(qs + swz_tc<TQ>(r, c), q + (size_t(start + q0 + r) * p.heads + h) * DK + c * 8);
       else
         *reinterpret_cast<uint4*>(q_tile + swz_tc<TQ>(r, c)) = make_uint4(0, 0, 0, 0);
     }
@@ -220,7 +226,7 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
 
   if (copy_warp) {
     // ------------------------------------------------------------ the thread that asks for the pages
-    // Page b goes into stage b % STAGES_TC as D / 64 boxes [64 keys x 64 dims] for K and for V, in
+    // Page b goes into stage b % STAGES_TC as DK / 64 and DV / 64 boxes [64 keys x 64 dims] for K and V, in
     // the swizzled layout; the stage's barrier counts the bytes. A stage is free again when the
     // O += P V that read it has completed (S of that page completed before it).
     // The first pages were asked for above; the rest is the first lane's alone.
@@ -241,22 +247,22 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     // ------------------------------------------------------------ the thread that issues matrix instructions
     if (lane == 0) {
       constexpr uint32_t IDESC_S = idesc_bf16(TQ, KEYS, false);
-      // all D dims of the output in one instruction: an instruction of M = 128, K = 16 takes 51 clocks at
+      // all DV dims of the output in one instruction: an instruction of M = 128, K = 16 takes 51 clocks at
       // least whatever its N (N / 2 clocks from N = 128 on), so their number is what a page costs
-      constexpr uint32_t IDESC_PV = idesc_bf16(TQ, D, true);
+      constexpr uint32_t IDESC_PV = idesc_bf16(TQ, DV, true);
       const uint64_t desc_q = smem_desc(smem_u32(q_tile), 16, 1024);
       const uint64_t desc_k0 = smem_desc(smem_u32(k_ring), 16, 1024);
       // V is MN-major: blocks of 64 dims lie KEYS * 128 bytes apart (the leading offset), groups of 8 keys
       // 1024 bytes (the stride offset)
       const uint64_t desc_v0 = smem_desc(smem_u32(v_ring), KEYS * 128, 1024);
-      constexpr uint64_t STAGE_UNITS = TILE_KV_BYTES >> 4;   // the address field counts 16-byte units
+      constexpr uint64_t K_UNITS = TILE_K_BYTES >> 4, V_UNITS = TILE_V_BYTES >> 4;   // the address field counts 16-byte units
       constexpr uint64_t Q_BLOCK = (TQ * 128) >> 4, KV_BLOCK = (KEYS * 128) >> 4;   // blocks of 64 dims
       // S_b = Q K_b^T into S buffer `buf`; the page sits in stage b % STAGES_TC
       auto issue_s = [&](int b, int buf) {
         const int st = b % STAGES_TC;
 #pragma unroll
-        for (int blk = 0; blk < D / 64; ++blk)
-          tc_mma4<2, 2>(tmem_base + buf * 64, desc_q + blk * Q_BLOCK, desc_k0 + st * STAGE_UNITS + blk * KV_BLOCK,
+        for (int blk = 0; blk < DK / 64; ++blk)
+          tc_mma4<2, 2>(tmem_base + buf * 64, desc_q + blk * Q_BLOCK, desc_k0 + st * K_UNITS + blk * KV_BLOCK,
                         IDESC_S, blk > 0 ? 1u : 0u);
         tc_commit(bar_s + buf * 8);
       };
@@ -280,7 +286,8 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
         if (alive) alive = mbar_wait(bar_p + buf * 8, phase, error_flag, 5);
         tc_fence_after();
         const int st = i % STAGES_TC;
-        tc_mma4_ts<128>(tmem_o, tmem_base + buf * 64, desc_v0 + st * STAGE_UNITS, IDESC_PV, i > 0 ? 1u : 0u);
+        tc_mma4_ts<128>(tmem_o, tmem_base + buf * 64, desc_v0 + st * V_UNITS, IDESC_PV, i > 0 ? 1u : 0u);
+        if (WIDE) tc_mma4_ts<128>(tmem_o, tmem_base + buf * 64 + KEYS / 2, desc_v0 + st * V_UNITS, IDESC_PV, 1u);
         tc_commit(bar_o + 8 * (i & 3));
         tc_commit(bar_free + 8 * st);   // the copy thread may refill this stage
         if (++buf == 3) { buf = 0; phase ^= 1; }
@@ -331,7 +338,7 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
         if (alive) alive = mbar_wait(bar_o + 8 * ((i - 1) & 3), ((i - 1) >> 2) & 1, error_flag, 2);
         tc_fence_after();
 #pragma unroll
-        for (int c0 = 0; c0 < D; c0 += 32) {
+        for (int c0 = 0; c0 < DV; c0 += 32) {
           float o[32];
           tmem_ld32(o_addr + c0, o);
 #pragma unroll
@@ -351,10 +358,20 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
         const float a = fast_exp2(x0), b = fast_exp2(x1);
         acc2[e & 3] = add2(acc2[e & 3], pack2(a, b));
         w[e] = pack_bf16(a, b);
+        if (WIDE) {      // what the rounding left, in the places of the two scores (a bfloat16's bits are a float32's upper half)
+          s[2 * e] = a - __uint_as_float(w[e] << 16);
+          s[2 * e + 1] = b - __uint_as_float(w[e] & 0xffff0000u);
+        }
       }
       // P in place of this page's S: keys 2c, 2c + 1 in column c of the buffer (this thread's row of S is in
       // registers since the load above)
       tmem_st_u32<KEYS / 2>(lane_addr + buf * 64, w);
+      if (WIDE) {
+        uint32_t lo[KEYS / 2];
+#pragma unroll
+        for (int e = 0; e < KEYS / 2; ++e) lo[e] = pack_bf16(s[2 * e], s[2 * e + 1]);
+        tmem_st_u32<KEYS / 2>(lane_addr + buf * 64 + KEYS / 2, lo);
+      }
       tmem_st_wait();
       float l0, l1, l2, l3;
       unpack2(add2(acc2[0], acc2[1]), l0, l1);
@@ -368,9 +385,9 @@ attention_tc_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __
     if (alive) alive = mbar_wait(bar_o + 8 * ((n_blocks - 1) & 3), ((n_blocks - 1) >> 2) & 1, error_flag, 3);
     tc_fence_after();
     const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-    __nv_bfloat16* dst = out + (size_t(start + q0 + row) * p.heads + h) * D;
+    __nv_bfloat16* dst = out + (size_t(start + q0 + row) * p.heads + h) * DV;
 #pragma unroll
-    for (int c0 = 0; c0 < D; c0 += 32) {
+    for (int c0 = 0; c0 < DV; c0 += 32) {
       float o[32];
       tmem_ld32(o_addr + c0, o);
       if (row_ok) {
@@ -788,25 +805,29 @@ static int g_pair_mode = 1;
 // they fill the device (the default), 2 = pairs wherever a K/V group has two heads or more
 PTB_API void ptb_attention_tc_pairs(int mode) { g_pair_mode = mode; }
 PTB_API int ptb_attention_tc_supports(int head_dim) { return (head_dim == 64 || head_dim == 128) ? 1 : 0; }
+// with key rows and value rows of different sizes
+PTB_API int ptb_attention_tc_supports_sizes(int head_dim, int v_dim) {
+  return ((head_dim == 64 || head_dim == 128) && v_dim == head_dim) || (head_dim == 192 && v_dim == 128) ? 1 : 0;
+}
 PTB_API int ptb_attention_tc_tile_tokens() { return TQ; }
 
 namespace {
-template <int D, bool BIAS>
+template <int DK, int DV, bool BIAS, bool WIDE>
 int launch_tc(const void* q, const void* k_pool, const void* v_pool, int pool_pages, void* out, const StepBatch& sb,
               const int* tile_seq, const int* tile_q0, int n_tiles, const TcParams& p, int* error_flag,
               cudaStream_t stream) {
-  const CUtensorMap* km = pool_map(k_pool, pool_pages, p.kv_heads, D);
-  const CUtensorMap* vm = pool_map(v_pool, pool_pages, p.kv_heads, D);
+  const CUtensorMap* km = pool_map(k_pool, pool_pages, p.kv_heads, DK);
+  const CUtensorMap* vm = pool_map(v_pool, pool_pages, p.kv_heads, DV);
   if (km == nullptr || vm == nullptr) return PTB_ERR_LAUNCH;
-  const size_t smem = 1024 + TQ * D * 2 + 2 * STAGES_TC * KEYS * D * 2 + 192;
+  const size_t smem = 1024 + TQ * DK * 2 + STAGES_TC * KEYS * (DK + DV) * 2 + 192;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(attention_tc_kernel<D, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) != cudaSuccess)
+    if (cudaFuncSetAttribute(attention_tc_kernel<DK, DV, BIAS, WIDE>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) != cudaSuccess)
       return PTB_ERR_LAUNCH;
     configured = true;
   }
   dim3 grid(p.heads, n_tiles);
-  attention_tc_kernel<D, BIAS><<<grid, BLOCK_THREADS, smem, stream>>>(
+  attention_tc_kernel<DK, DV, BIAS, WIDE><<<grid, BLOCK_THREADS, smem, stream>>>(
       (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_pool, (const __nv_bfloat16*)v_pool, (__nv_bfloat16*)out, sb,
       tile_seq, tile_q0, p, *km, *vm, error_flag);
   return launch_status();
@@ -814,24 +835,30 @@ int launch_tc(const void* q, const void* k_pool, const void* v_pool, int pool_pa
 }  // namespace
 
 // Causal attention of prompt tiles of 128 tokens (tile_seq / tile_q0 as for the other attention
-// kernels, 128 tokens per tile), bfloat16, head size 64 or 128, no window. k_pool / v_pool: the pools of
-// one cache entry, [pool_pages][kv_heads][64][head_dim]. `slopes`: per-head score
-// slopes [heads] float32 (already rounded to bfloat16 values), or null. `error_flag` is a device int
-// that stays 0 unless a bounded wait inside the kernel ran out.
-PTB_API int ptb_attention_tc(const void* q, const void* k_pool, const void* v_pool, int pool_pages, void* out,
-                             const StepBatch* sb,
-                             const int* tile_seq, const int* tile_q0, int n_tiles, const float* slopes, int heads,
-                             int kv_heads, int head_dim, float scale, int* error_flag, cudaStream_t stream) {
+// kernels, 128 tokens per tile), bfloat16, no window. Keys of head_dim and values of v_dim entries: 64 or 128 alike,
+// or 192 beside 128. k_pool / v_pool: the pools of one cache entry, [pool_pages][kv_heads][64][head_dim or v_dim].
+// `slopes`: per-head score slopes [heads] float32 (already rounded to bfloat16 values), or null. wide_weights: the
+// softmax weights meet the values as two bfloat16 terms. `error_flag` is a device int that stays 0 unless a
+// bounded wait inside the kernel ran out.
+PTB_API int ptb_attention_tc_sizes(const void* q, const void* k_pool, const void* v_pool, int pool_pages, void* out,
+                                   const StepBatch* sb, const int* tile_seq, const int* tile_q0, int n_tiles,
+                                   const float* slopes, int heads, int kv_heads, int head_dim, int v_dim, float scale,
+                                   int wide_weights, int* error_flag, cudaStream_t stream) {
   if (n_tiles <= 0) return PTB_OK;
   if (pool_pages <= 0 || (reinterpret_cast<uintptr_t>(k_pool) | reinterpret_cast<uintptr_t>(v_pool)) & 15) return PTB_ERR_ALIGN;
-  if ((head_dim != 64 && head_dim != 128) || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 || n_tiles > 65535 ||
-      error_flag == nullptr)
+  if (!ptb_attention_tc_supports_sizes(head_dim, v_dim) || heads <= 0 || kv_heads <= 0 || heads % kv_heads != 0 ||
+      n_tiles > 65535 || error_flag == nullptr)
     return PTB_ERR_SIZE;
   TcParams p;
   p.heads = heads; p.kv_heads = kv_heads; p.scale = scale; p.slopes = slopes;
-  if (head_dim == 64)
-    return slopes ? launch_tc<64, true>(q, k_pool, v_pool, pool_pages, out, *sb, tile_seq, tile_q0, n_tiles, p, error_flag, stream)
-                  : launch_tc<64, false>(q, k_pool, v_pool, pool_pages, out, *sb, tile_seq, tile_q0, n_tiles, p, error_flag, stream);
+#define PTB_TC(DK, DV, B, W) \
+  launch_tc<DK, DV, B, W>(q, k_pool, v_pool, pool_pages, out, *sb, tile_seq, tile_q0, n_tiles, p, error_flag, stream)
+  if (wide_weights) {
+    if (slopes) return PTB_ERR_SIZE;      // not built: no model has score slopes beside split weights
+    return head_dim == 64 ? PTB_TC(64, 64, false, true) : head_dim == 128 ? PTB_TC(128, 128, false, true) : PTB_TC(192, 128, false, true);
+  }
+  if (head_dim == 192) return slopes ? PTB_ERR_SIZE : PTB_TC(192, 128, false, false);
+  if (head_dim == 64) return slopes ? PTB_TC(64, 64, true, false) : PTB_TC(64, 64, false, false);
   // Head size 128 leaves room for one block an SM: two heads of a K/V group share a block, with keys in
   // steps of two pages, where a group has two heads or more and the pairs fill the device. (With head size
   // 64 two blocks of the kernel above share an SM, each with three S buffers, and are a quarter faster than
@@ -841,6 +868,15 @@ PTB_API int ptb_attention_tc(const void* q, const void* k_pool, const void* v_po
   if (qpk >= 2 && g_pair_mode != 0 && (pair_blocks >= sm_count() || g_pair_mode == 2))
     return slopes ? launch_tc_pair<128, true>(q, k_pool, v_pool, pool_pages, out, *sb, tile_seq, tile_q0, n_tiles, p, error_flag, stream)
                   : launch_tc_pair<128, false>(q, k_pool, v_pool, pool_pages, out, *sb, tile_seq, tile_q0, n_tiles, p, error_flag, stream);
-  return slopes ? launch_tc<128, true>(q, k_pool, v_pool, pool_pages, out, *sb, tile_seq, tile_q0, n_tiles, p, error_flag, stream)
-                : launch_tc<128, false>(q, k_pool, v_pool, pool_pages, out, *sb, tile_seq, tile_q0, n_tiles, p, error_flag, stream);
+  return slopes ? PTB_TC(128, 128, true, false) : PTB_TC(128, 128, false, false);
+#undef PTB_TC
+}
+
+PTB_API int ptb_attention_tc(const void* q, const void* k_pool, const void* v_pool, int pool_pages, void* out,
+                             const StepBatch* sb,
+                             const int* tile_seq, const int* tile_q0, int n_tiles, const float* slopes, int heads,
+                             int kv_heads, int head_dim, float scale, int* error_flag, cudaStream_t stream) {
+  if (!ptb_attention_tc_supports(head_dim)) return PTB_ERR_SIZE;
+  return ptb_attention_tc_sizes(q, k_pool, v_pool, pool_pages, out, sb, tile_seq, tile_q0, n_tiles, slopes, heads, kv_heads,
+                                head_dim, head_dim, scale, 0, error_flag, stream);
 }

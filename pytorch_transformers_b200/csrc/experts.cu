@@ -7,6 +7,8 @@
 // are chosen (ties: lowest index); the weight of a chosen output is s * route_scale (not renormalised).
 // The last n - n_experts outputs are identity experts: they pass their input on.
 // score_kind 1: s = sigmoid(z) per output instead of the softmax. correction may be null (none).
+// score_kind 2: the choice is by the logits z (+ correction) themselves, and the weights are the softmax over the
+// chosen logits alone, times route_scale. A bias per output may be part of the logits: z = W_r h + bias.
 #include "common.cuh"
 
 namespace {
@@ -20,8 +22,8 @@ constexpr int ROUTE_TOKENS = 8;   // tokens of a block of the logits kernel for 
 // block; a token's sums have one fixed order whatever else is in the batch.
 template <typename T, int TPB>
 __global__ void __launch_bounds__(32 * ROUTE_WARPS)
-route_logits_kernel(const T* __restrict__ h, const float* __restrict__ w_router, float* __restrict__ z, int n_tokens,
-                    int width, int n) {
+route_logits_kernel(const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ bias,
+                    float* __restrict__ z, int n_tokens, int width, int n, int n_bias) {
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
   const int t0 = blockIdx.x * TPB, e = blockIdx.y * ROUTE_WARPS + warp;
   if (e >= n) return;
@@ -41,7 +43,7 @@ route_logits_kernel(const T* __restrict__ h, const float* __restrict__ w_router,
   }
 #pragma unroll
   for (int i = 0; i < TPB; ++i) {
-    const float v = warp_sum(d[i]);
+    const float v = warp_sum(d[i]) + (bias != nullptr && e < n_bias ? bias[e] : 0.f);
     if (lane == 0 && t0 + i < n_tokens) z[size_t(t0 + i) * n + e] = v;
   }
 }
@@ -79,6 +81,7 @@ route_select_kernel(const float* __restrict__ zs_all, const float* __restrict__ 
   for (int v = 0; v < ROUTE_VPL; ++v) {
     const int e = lane + 32 * v;
     if (score_kind == 1) s[v] = (e < n) ? 1.f / (1.f + expf(-z[v])) : 0.f;
+    else if (score_kind == 2) s[v] = (e < n) ? z[v] : 0.f;
     else s[v] = s[v] / sum;
     if (e < n) choice[e] = s[v] + (correction ? correction[e] : 0.f);
   }
@@ -148,15 +151,23 @@ route_select_kernel(const float* __restrict__ zs_all, const float* __restrict__ 
           open[u] = false;
         }
       ids[size_t(t) * top + k] = best_e;
-      if (!normalize) gates[size_t(t) * top + k] = sv * route_scale;
+      if (!normalize && score_kind != 2) gates[size_t(t) * top + k] = sv * route_scale;
     }
-    if (normalize) {
+    if (normalize || score_kind == 2) {
       sv = __shfl_sync(0xffffffffu, sv, best_e % 32);
       chosen_sum += sv;
       if (lane == 0) gates[size_t(t) * top + k] = sv;
     }
   }
-  if (normalize && lane == 0) {
+  if (score_kind == 2) {
+    if (lane == 0) {      // the chosen logits wait in `gates`, in the order of the choice
+      float* mine = gates + size_t(t) * top;
+      float m = -INFINITY, total = 0.f;
+      for (int k = 0; k < top; ++k) m = fmaxf(m, mine[k]);
+      for (int k = 0; k < top; ++k) total += expf(mine[k] - m);
+      for (int k = 0; k < top; ++k) mine[k] = expf(mine[k] - m) / total * route_scale;
+    }
+  } else if (normalize && lane == 0) {
     // weights = scores / (their sum + 1e-20) * scale
     const float total = chosen_sum + 1e-20f;
     for (int k = 0; k < top; ++k) gates[size_t(t) * top + k] = gates[size_t(t) * top + k] / total * route_scale;
@@ -354,18 +365,20 @@ int launch_expert_linear(const void* x, const void* w, void* out, const int* pla
 // `logits`: float32 [n_tokens, n + extra]: the router matrix has `extra` more rows whose logits are formed with the
 // others and take no part in the choice (a gate that reads the same input). group_top 1 or 2: a group is scored by its
 // largest choice score or by the sum of its two largest. normalize: weights = scores / (sum of the chosen + 1e-20) * scale.
-PTB_API int ptb_route_grouped(int dtype, const void* h, const float* w_router, const float* correction, float* logits, int* ids,
+// bias: [n] float32 or null. score_kind: 0 softmax, 1 sigmoid, 2 the logits with a softmax over the chosen.
+PTB_API int ptb_route_biased(int dtype, const void* h, const float* w_router, const float* bias, const float* correction,
+                             float* logits, int* ids,
                       float* gates, int n_tokens, int width, int n, int n_groups, int keep, int top, float route_scale,
                       int score_kind, int extra, int group_top, int normalize, cudaStream_t stream) {
   if (n_tokens <= 0) return PTB_OK;
   if (n <= 0 || n > 32 * ROUTE_VPL || n_groups <= 0 || n % n_groups != 0 || keep <= 0 || keep > n_groups || top <= 0 ||
-      top > (n / n_groups) * keep || width <= 0 || score_kind < 0 || score_kind > 1 || extra < 0 || group_top < 1 || group_top > 2)
+      top > (n / n_groups) * keep || width <= 0 || score_kind < 0 || score_kind > 2 || extra < 0 || group_top < 1 || group_top > 2)
     return PTB_ERR_SIZE;
   // few tokens (steps of single tokens): one token a block, so that the blocks fill the device
   const int tpb = n_tokens >= 2 * sm_count() ? ROUTE_TOKENS : 1;
   dim3 grid((n_tokens + tpb - 1) / tpb, (n + extra + ROUTE_WARPS - 1) / ROUTE_WARPS);
 #define PTB_ROUTE(TT, NTOK) \
-  route_logits_kernel<TT, NTOK><<<grid, 32 * ROUTE_WARPS, 0, stream>>>((const TT*)h, w_router, logits, n_tokens, width, n + extra)
+  route_logits_kernel<TT, NTOK><<<grid, 32 * ROUTE_WARPS, 0, stream>>>((const TT*)h, w_router, bias, logits, n_tokens, width, n + extra, n)
   if (dtype == PTB_F32) {
     if (tpb == 1) PTB_ROUTE(float, 1);
     else PTB_ROUTE(float, ROUTE_TOKENS);
@@ -381,6 +394,13 @@ PTB_API int ptb_route_grouped(int dtype, const void* h, const float* w_router, c
   route_select_kernel<<<(n_tokens + ROUTE_WARPS - 1) / ROUTE_WARPS, 32 * ROUTE_WARPS, smem, stream>>>(
       logits, correction, ids, gates, n_tokens, n, n_groups, keep, top, route_scale, score_kind, n + extra, group_top, normalize);
   return launch_status();
+}
+
+PTB_API int ptb_route_grouped(int dtype, const void* h, const float* w_router, const float* correction, float* logits, int* ids,
+                              float* gates, int n_tokens, int width, int n, int n_groups, int keep, int top, float route_scale,
+                              int score_kind, int extra, int group_top, int normalize, cudaStream_t stream) {
+  return ptb_route_biased(dtype, h, w_router, nullptr, correction, logits, ids, gates, n_tokens, width, n, n_groups, keep, top,
+                          route_scale, score_kind, extra, group_top, normalize, stream);
 }
 
 PTB_API int ptb_route(int dtype, const void* h, const float* w_router, const float* correction, float* logits, int* ids,

@@ -7,7 +7,7 @@
 //           of the same columns; out[row, f] = silu(gate) * up, bfloat16.
 //   mode 1: x rows are the sorted rows themselves; out[row, n] float32.
 //   mode 2: x rows gathered as in mode 0, 128 plain matrix rows; out[row, n] = act(row_scale[pair] * sum), bfloat16
-//           (an expert without a gate whose input is the token's row times the pair's weight).
+//           (an expert without a gate; with row_scale its input is the token's row times the pair's weight).
 // A row's sums do not depend on its place in a tile or on the other rows.
 #include "mma_common.cuh"
 

@@ -56,14 +56,15 @@ __global__ void latent_store_kernel(const T* __restrict__ src, long long src_str
 // One block = one tile (tile_tokens consecutive new tokens of a sequence) x one chunk of
 // heads_per_block heads x one split of the key pages; tile_tokens * heads_per_block <= ROWS.
 //   q_abs [tokens, heads, rank] float32: queries with the key up-projection folded in
-//   q     [tokens, heads, q_dim]: the projection's rows; the part to rotate starts at q_rot_off
+//   q     [tokens, heads, q_dim] (tokens q_stride entries apart): the projection's rows; the part to rotate
+//         starts at q_rot_off
 //   pool  [pages][64][rank + rot_dim]
 //   out   [tokens, heads, rank]: softmax-weighted sums of the latents
 // With n_splits > 1 a block writes (max, sum, unnormalised sums) of its pages to `part` and
 // latent_join_kernel merges the splits in order.
 template <typename T, int DPT>
 __global__ void __launch_bounds__(THREADS)
-latent_attention_kernel(const float* __restrict__ q_abs, const T* __restrict__ q, int q_dim, int q_rot_off,
+latent_attention_kernel(const float* __restrict__ q_abs, const T* __restrict__ q, long long q_stride, int q_dim, int q_rot_off,
                         const T* __restrict__ pool, float* __restrict__ part, T* __restrict__ out, StepBatch sb,
                         const int* __restrict__ tile_seq, const int* __restrict__ tile_q0,
                         const float* __restrict__ rope_cos, const float* __restrict__ rope_sin, int rot_pairs,
@@ -96,7 +97,7 @@ latent_attention_kernel(const float* __restrict__ q_abs, const T* __restrict__ q
     const int ti = rr / heads_per_block, hh = h0 + rr % heads_per_block;
     const bool ok = ti < toks && hh < heads && rr < tile_tokens * heads_per_block;
     const size_t tok = size_t(start + q0 + ti);
-    const T* src = q + (tok * heads + hh) * q_dim + q_rot_off;
+    const T* src = q + tok * q_stride + size_t(hh) * q_dim + q_rot_off;
     float* dst = qs + rr * qstride + rank;
     if (e < rot_pairs) {
       const int ia = interleaved ? 2 * e : e, ib = interleaved ? 2 * e + 1 : e + rot_pairs;
@@ -260,7 +261,7 @@ __global__ void latent_join_kernel(const float* __restrict__ part, T* __restrict
 }
 
 template <typename T, int DPT>
-int launch_latent(const float* q_abs, const void* q, int q_dim, int q_rot_off, const void* pool, float* part,
+int launch_latent(const float* q_abs, const void* q, long long q_stride, int q_dim, int q_rot_off, const void* pool, float* part,
                   void* out, const StepBatch& sb, const int* tile_seq, const int* tile_q0, int n_tiles,
                   const float* rope_cos, const float* rope_sin, int rot_pairs, int interleaved, int heads, int rank,
                   int rot_dim, int tile_tokens, int heads_per_block, float scale, int n_splits, cudaStream_t stream) {
@@ -277,7 +278,7 @@ int launch_latent(const float* q_abs, const void* q, int q_dim, int q_rot_off, c
   const int chunks = (heads + heads_per_block - 1) / heads_per_block;
   dim3 grid(n_tiles, chunks, n_splits);
   latent_attention_kernel<T, DPT><<<grid, THREADS, smem, stream>>>(
-      q_abs, (const T*)q, q_dim, q_rot_off, (const T*)pool, part, (T*)out, sb, tile_seq, tile_q0, rope_cos, rope_sin,
+      q_abs, (const T*)q, q_stride, q_dim, q_rot_off, (const T*)pool, part, (T*)out, sb, tile_seq, tile_q0, rope_cos, rope_sin,
       rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens, heads_per_block, scale, n_splits);
   int rc = launch_status();
   if (rc != PTB_OK || n_splits <= 1) return rc;
@@ -287,13 +288,13 @@ int launch_latent(const float* q_abs, const void* q, int q_dim, int q_rot_off, c
 }
 
 template <typename T>
-int dispatch_latent(const float* q_abs, const void* q, int q_dim, int q_rot_off, const void* pool, float* part,
+int dispatch_latent(const float* q_abs, const void* q, long long q_stride, int q_dim, int q_rot_off, const void* pool, float* part,
                     void* out, const StepBatch& sb, const int* tile_seq, const int* tile_q0, int n_tiles,
                     const float* rope_cos, const float* rope_sin, int rot_pairs, int interleaved, int heads, int rank,
                     int rot_dim, int tile_tokens, int heads_per_block, float scale, int n_splits,
                     cudaStream_t stream) {
 #define PTB_LATENT(D)                                                                                             \
-  return launch_latent<T, D>(q_abs, q, q_dim, q_rot_off, pool, part, out, sb, tile_seq, tile_q0, n_tiles, rope_cos, \
+  return launch_latent<T, D>(q_abs, q, q_stride, q_dim, q_rot_off, pool, part, out, sb, tile_seq, tile_q0, n_tiles, rope_cos, \
                              rope_sin, rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens, heads_per_block,  \
                              scale, n_splits, stream)
   if (rank <= 64) PTB_LATENT(8);
@@ -333,7 +334,7 @@ PTB_API int ptb_latent_store(int dtype, const void* src, long long src_stride, c
   return launch_status();
 }
 
-PTB_API int ptb_latent_attention(int dtype, const float* q_abs, const void* q, int q_dim, int q_rot_off,
+PTB_API int ptb_latent_attention(int dtype, const float* q_abs, const void* q, long long q_stride, int q_dim, int q_rot_off,
                                  const void* pool, float* part, void* out, const StepBatch* sb, const int* tile_seq,
                                  const int* tile_q0, int n_tiles, const float* rope_cos, const float* rope_sin,
                                  int rot_pairs, int interleaved, int heads, int rank, int rot_dim, int tile_tokens,
@@ -346,26 +347,28 @@ PTB_API int ptb_latent_attention(int dtype, const float* q_abs, const void* q, i
   if (n_splits > 1 && part == nullptr) return PTB_ERR_SIZE;
   if (rot_pairs > 0 && (rope_cos == nullptr || rope_sin == nullptr)) return PTB_ERR_SIZE;
   if (dtype == PTB_F32)
-    return dispatch_latent<float>(q_abs, q, q_dim, q_rot_off, pool, part, out, *sb, tile_seq, tile_q0, n_tiles,
+    return dispatch_latent<float>(q_abs, q, q_stride, q_dim, q_rot_off, pool, part, out, *sb, tile_seq, tile_q0, n_tiles,
                                   rope_cos, rope_sin, rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens,
                                   heads_per_block, scale, n_splits, stream);
   if (dtype == PTB_BF16)
-    return dispatch_latent<__nv_bfloat16>(q_abs, q, q_dim, q_rot_off, pool, part, out, *sb, tile_seq, tile_q0, n_tiles,
+    return dispatch_latent<__nv_bfloat16>(q_abs, q, q_stride, q_dim, q_rot_off, pool, part, out, *sb, tile_seq, tile_q0, n_tiles,
                                           rope_cos, rope_sin, rot_pairs, interleaved, heads, rank, rot_dim,
                                           tile_tokens, heads_per_block, scale, n_splits, stream);
   return PTB_ERR_DTYPE;
 }
 
 // ------------------------------------------------------------------------------------------------
-// The same attention in bfloat16 on the tensor cores (mma.m16n8k16, float32 sums), for rank a multiple
-// of 64 and rot_dim a multiple of 16. A block of 4 warps takes the 16 rows of a tile (the heads of a
+// The same attention in bfloat16 on the tensor cores (mma.m16n8k16, float32 sums), for rank and rot_dim
+// multiples of 16. A block of 4 warps takes the 16 rows of a tile (the heads of a
 // token in a step of single tokens) and walks its share of the key pages. A page [64][rank + rot_dim]
 // comes into shared memory once (cp.async, rows 16 bytes apart from a multiple of 128 so that ldmatrix
 // meets no bank twice) and serves both products, for up to four groups of 4 warps with 16 rows each (a tile of a
 // prompt is 16 tokens x 4 heads, so that a staged page meets 64 rows): warp w of a group forms the scores of keys 16 w .. 16 w + 15
 // (S = Q K^T over all rank + rot_dim entries), the warps exchange row maxima and sums through shared
-// memory, the weights go to shared memory as bfloat16, and warp w adds P V for the columns
-// w rank / 4 .. (w + 1) rank / 4 of the output, V being the first `rank` entries of the same rows.
+// memory, the weights go to shared memory as bfloat16, and warp w adds P V for a quarter of the output's
+// columns (in whole groups of 16; the last warps have fewer, or none, where rank is no multiple of 64), V being
+// the first `rank` entries of the same rows. With WIDE the weights meet V as two bfloat16 terms (the rounded
+// weight and what the rounding left: 16 bits of mantissa) and their sum is formed from the float32 weights.
 // The query rows are rounded to bfloat16 once (q_abs comes in float32); scores, maxima, sums and the
 // output sums are float32. Splits and their join are those of the general kernel.
 #include "mma_common.cuh"
@@ -374,12 +377,12 @@ namespace {
 
 constexpr int MTHREADS = 128;
 
-// NF: 8-column fragments of the output per warp (rank = 32 NF). TG: groups of 4 warps; every group has 16
+// NF: 8-column fragments of the output per warp (4 warps cover rank <= 32 NF columns). TG: groups of 4 warps; every group has 16
 // rows of the tile (a tile of a prompt holds 16 TG rows: tokens x heads), and all groups use one staged page.
-template <int NF, int TG>
+template <int NF, int TG, bool WIDE>
 __global__ void __launch_bounds__(MTHREADS * TG)
-latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16* __restrict__ q, int q_dim,
-                            int q_rot_off, const __nv_bfloat16* __restrict__ pool, float* __restrict__ part,
+latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16* __restrict__ q, long long q_stride,
+                            int q_dim, int q_rot_off, const __nv_bfloat16* __restrict__ pool, float* __restrict__ part,
                             __nv_bfloat16* __restrict__ out, StepBatch sb, const int* __restrict__ tile_seq,
                             const int* __restrict__ tile_q0, const float* __restrict__ rope_cos,
                             const float* __restrict__ rope_sin, int rot_pairs, int interleaved, int heads, int rank,
@@ -390,8 +393,9 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
   const int rowb = dk * 2 + 16;                       // bytes of a staged row
   unsigned char* q_s = msm;                           // [16 TG][rowb]
   unsigned char* k_s = q_s + QROWS * rowb;            // [64][rowb]
+  constexpr int P_BYTES = (WIDE ? 2 : 1) * 16 * 144;  // a group's weights; with WIDE their second terms behind them
   unsigned char* p_all = k_s + PTB_PAGE * rowb;       // [TG][16][144]: 64 weights and 16 bytes of padding a row
-  float* wmax_all = reinterpret_cast<float*>(p_all + TG * 16 * 144);   // [TG][4][16]
+  float* wmax_all = reinterpret_cast<float*>(p_all + TG * P_BYTES);     // [TG][4][16]
   float* wsum_all = wmax_all + TG * 64;                                 // [TG][4][16]
 
   const int tile = blockIdx.x, h0 = blockIdx.y * heads_per_block, split = blockIdx.z;
@@ -401,7 +405,7 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
   const int tid = threadIdx.x, lane = tid % 32;
   const int tg = tid / MTHREADS, warp = (tid / 32) % 4;      // group of warps, warp in the group
   const int used_rows = tile_tokens * heads_per_block;
-  unsigned char* p_s = p_all + tg * 16 * 144;
+  unsigned char* p_s = p_all + tg * P_BYTES;
   float* wmax = wmax_all + tg * 64;
   float* wsum = wsum_all + tg * 64;
 
@@ -419,7 +423,7 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
     const int ti = rr / heads_per_block, hh = h0 + rr % heads_per_block;
     const bool ok = ti < toks && hh < heads && rr < used_rows;
     const size_t tok = size_t(start + q0 + ti);
-    const __nv_bfloat16* src = q + (tok * heads + hh) * q_dim + q_rot_off;
+    const __nv_bfloat16* src = q + tok * q_stride + size_t(hh) * q_dim + q_rot_off;
     __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(q_s + rr * rowb) + rank;
     if (e < rot_pairs) {
       const int ia = interleaved ? 2 * e : e, ib = interleaved ? 2 * e + 1 : e + rot_pairs;
@@ -457,6 +461,7 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
   const int chunks = dk / 8;
   const uint32_t q_base = smem_u32(q_s) + tg * 16 * rowb, k_base = smem_u32(k_s), p_base = smem_u32(p_s);
   const int col0 = warp * NF * 8;       // first output column of this warp
+  const int my_pairs = min(NF / 2, max(0, rank - col0) / 16);   // groups of 16 columns that this warp has
 
   for (int kb = kb_lo; kb <= kb_hi; ++kb) {
     const __nv_bfloat16* kp = pool + kv_offset(pages[kb], 0, 0, 1, dk);
@@ -519,9 +524,16 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
         const float p1 = (s[f][hf * 2 + 1] == -INFINITY) ? 0.f : expf(s[f][hf * 2 + 1] - m_new[hf]);
         // the weights as the second product sees them, and their sum from the same rounded values
         const __nv_bfloat162 pr = __floats2bfloat162_rn(p0, p1);
-        sum[hf] += __bfloat162float(pr.x) + __bfloat162float(pr.y);
         const int rr = hf ? r_hi : r_lo;
-        *reinterpret_cast<__nv_bfloat162*>(p_s + rr * 144 + (warp * 16 + f * 8 + (lane % 4) * 2) * 2) = pr;
+        unsigned char* at = p_s + rr * 144 + (warp * 16 + f * 8 + (lane % 4) * 2) * 2;
+        *reinterpret_cast<__nv_bfloat162*>(at) = pr;
+        const float h0f = __bfloat162float(pr.x), h1f = __bfloat162float(pr.y);
+        if (WIDE) {
+          sum[hf] += p0 + p1;
+          *reinterpret_cast<__nv_bfloat162*>(at + 16 * 144) = __floats2bfloat162_rn(p0 - h0f, p1 - h1f);
+        } else {
+          sum[hf] += h0f + h1f;
+        }
       }
 #pragma unroll
     for (int hf = 0; hf < 2; ++hf) {
@@ -549,16 +561,22 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
     // O += P V for this warp's columns
 #pragma unroll
     for (int ks = 0; ks < PTB_PAGE / 16; ++ks) {
-      uint32_t a[4];
+      uint32_t a[4], lo[4];
       ldmatrix_x4(a[0], a[1], a[2], a[3], p_base + (lane & 15) * 144 + (ks * 2 + (lane >> 4)) * 16);
+      if (WIDE) ldmatrix_x4(lo[0], lo[1], lo[2], lo[3], p_base + 16 * 144 + (lane & 15) * 144 + (ks * 2 + (lane >> 4)) * 16);
       const int id = lane >> 3;
 #pragma unroll
       for (int jp = 0; jp < NF / 2; ++jp) {
+        if (jp >= my_pairs) continue;      // the same for the whole warp
         uint32_t b0, b1, b2, b3;
         ldmatrix_x4_trans(b0, b1, b2, b3,
                           k_base + (ks * 16 + (id & 1) * 8 + (lane & 7)) * rowb + (col0 + jp * 16 + (id >> 1) * 8) * 2);
         mma_bf16(acc[2 * jp], a, b0, b1);
         mma_bf16(acc[2 * jp + 1], a, b2, b3);
+        if (WIDE) {
+          mma_bf16(acc[2 * jp], lo, b0, b1);
+          mma_bf16(acc[2 * jp + 1], lo, b2, b3);
+        }
       }
     }
   }
@@ -575,6 +593,7 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
       }
 #pragma unroll
       for (int j = 0; j < NF; ++j) {
+        if (j >= 2 * my_pairs) continue;
         p[2 + col0 + j * 8 + c0] = acc[j][hf * 2];
         p[2 + col0 + j * 8 + c0 + 1] = acc[j][hf * 2 + 1];
       }
@@ -584,29 +603,30 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
       __nv_bfloat16* o = out + (size_t(start + q0 + ti) * heads + hh) * rank + col0;
 #pragma unroll
       for (int j = 0; j < NF; ++j)
-        *reinterpret_cast<__nv_bfloat162*>(o + j * 8 + c0) = __floats2bfloat162_rn(acc[j][hf * 2] * inv, acc[j][hf * 2 + 1] * inv);
+        if (j < 2 * my_pairs)
+          *reinterpret_cast<__nv_bfloat162*>(o + j * 8 + c0) = __floats2bfloat162_rn(acc[j][hf * 2] * inv, acc[j][hf * 2 + 1] * inv);
     }
   }
 }
 
-template <int NF, int TG>
-int launch_latent_mma_tg(const float* q_abs, const void* q, int q_dim, int q_rot_off, const void* pool, float* part,
+template <int NF, int TG, bool WIDE>
+int launch_latent_mma_tg(const float* q_abs, const void* q, long long q_stride, int q_dim, int q_rot_off, const void* pool, float* part,
                          void* out, const StepBatch& sb, const int* tile_seq, const int* tile_q0, int n_tiles,
                          const float* rope_cos, const float* rope_sin, int rot_pairs, int interleaved, int heads, int rank,
                          int rot_dim, int tile_tokens, int heads_per_block, float scale, int n_splits, cudaStream_t stream) {
   const int rowb = (rank + rot_dim) * 2 + 16;
-  const size_t smem = size_t(16 * TG + PTB_PAGE) * rowb + TG * (16 * 144 + 2 * 64 * sizeof(float));
+  const size_t smem = size_t(16 * TG + PTB_PAGE) * rowb + TG * ((WIDE ? 2 : 1) * 16 * 144 + 2 * 64 * sizeof(float));
   if (smem > 220 * 1024) return PTB_ERR_SIZE;
   static size_t configured = 48 * 1024;
   if (smem > configured) {
-    if (cudaFuncSetAttribute(latent_attention_mma_kernel<NF, TG>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) !=
+    if (cudaFuncSetAttribute(latent_attention_mma_kernel<NF, TG, WIDE>, cudaFuncAttributeMaxDynamicSharedMemorySize, int(smem)) !=
         cudaSuccess)
       return PTB_ERR_LAUNCH;
     configured = smem;
   }
   const int chunks = (heads + heads_per_block - 1) / heads_per_block;
-  latent_attention_mma_kernel<NF, TG><<<dim3(n_tiles, chunks, n_splits), MTHREADS * TG, smem, stream>>>(
-      q_abs, (const __nv_bfloat16*)q, q_dim, q_rot_off, (const __nv_bfloat16*)pool, part, (__nv_bfloat16*)out, sb,
+  latent_attention_mma_kernel<NF, TG, WIDE><<<dim3(n_tiles, chunks, n_splits), MTHREADS * TG, smem, stream>>>(
+      q_abs, (const __nv_bfloat16*)q, q_stride, q_dim, q_rot_off, (const __nv_bfloat16*)pool, part, (__nv_bfloat16*)out, sb,
       tile_seq, tile_q0, rope_cos, rope_sin, rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens, heads_per_block,
       scale, n_splits);
   int rc = launch_status();
@@ -616,14 +636,14 @@ int launch_latent_mma_tg(const float* q_abs, const void* q, int q_dim, int q_rot
   return launch_status();
 }
 
-template <int NF>
-int launch_latent_mma(const float* q_abs, const void* q, int q_dim, int q_rot_off, const void* pool, float* part,
+template <int NF, bool WIDE>
+int launch_latent_mma(const float* q_abs, const void* q, long long q_stride, int q_dim, int q_rot_off, const void* pool, float* part,
                       void* out, const StepBatch& sb, const int* tile_seq, const int* tile_q0, int n_tiles,
                       const float* rope_cos, const float* rope_sin, int rot_pairs, int interleaved, int heads, int rank,
                       int rot_dim, int tile_tokens, int heads_per_block, float scale, int n_splits, cudaStream_t stream) {
   const int rows = tile_tokens * heads_per_block;
 #define PTB_LTG(TGV)                                                                                                  \
-  return launch_latent_mma_tg<NF, TGV>(q_abs, q, q_dim, q_rot_off, pool, part, out, sb, tile_seq, tile_q0, n_tiles,     \
+  return launch_latent_mma_tg<NF, TGV, WIDE>(q_abs, q, q_stride, q_dim, q_rot_off, pool, part, out, sb, tile_seq, tile_q0, n_tiles,     \
                                        rope_cos, rope_sin, rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens,   \
                                        heads_per_block, scale, n_splits, stream)
   if (rows <= 16) PTB_LTG(1);
@@ -636,14 +656,16 @@ int launch_latent_mma(const float* q_abs, const void* q, int q_dim, int q_rot_of
 }  // namespace
 
 PTB_API int ptb_latent_attention_mma_supports(int rank, int rot_dim) {
-  return rank > 0 && rank <= 512 && rank % 64 == 0 && rot_dim >= 0 && rot_dim % 16 == 0;
+  return rank > 0 && rank <= 512 && rank % 16 == 0 && rot_dim >= 0 && rot_dim % 16 == 0;
 }
 
-PTB_API int ptb_latent_attention_mma(const float* q_abs, const void* q, int q_dim, int q_rot_off, const void* pool,
+// wide_weights: the softmax weights as two bfloat16 terms
+PTB_API int ptb_latent_attention_mma(const float* q_abs, const void* q, long long q_stride, int q_dim, int q_rot_off, const void* pool,
                                      float* part, void* out, const StepBatch* sb, const int* tile_seq,
                                      const int* tile_q0, int n_tiles, const float* rope_cos, const float* rope_sin,
                                      int rot_pairs, int interleaved, int heads, int rank, int rot_dim, int tile_tokens,
-                                     int heads_per_block, float scale, int n_splits, cudaStream_t stream) {
+                                     int heads_per_block, float scale, int n_splits, int wide_weights,
+                                     cudaStream_t stream) {
   if (n_tiles <= 0) return PTB_OK;
   if (!ptb_latent_attention_mma_supports(rank, rot_dim) || heads <= 0 || rot_pairs < 0 || 2 * rot_pairs > rot_dim ||
       tile_tokens <= 0 || heads_per_block <= 0 || tile_tokens * heads_per_block > 4 * ROWS || n_splits < 1 ||
@@ -652,11 +674,16 @@ PTB_API int ptb_latent_attention_mma(const float* q_abs, const void* q, int q_di
   if (n_splits > 1 && part == nullptr) return PTB_ERR_SIZE;
   if (rot_pairs > 0 && (rope_cos == nullptr || rope_sin == nullptr)) return PTB_ERR_SIZE;
   if (!aligned16(pool) || !aligned16(out)) return PTB_ERR_ALIGN;
-#define PTB_LMMA(NFV)                                                                                               \
-  return launch_latent_mma<NFV>(q_abs, q, q_dim, q_rot_off, pool, part, out, *sb, tile_seq, tile_q0, n_tiles, rope_cos, \
-                                rope_sin, rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens, heads_per_block,   \
-                                scale, n_splits, stream)
-  switch (rank / 64) {
+#define PTB_LMMA1(NFV, W)                                                                                              \
+  return launch_latent_mma<NFV, W>(q_abs, q, q_stride, q_dim, q_rot_off, pool, part, out, *sb, tile_seq, tile_q0, n_tiles, \
+                                   rope_cos, rope_sin, rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens,        \
+                                   heads_per_block, scale, n_splits, stream)
+#define PTB_LMMA(NFV)                      \
+  do {                                     \
+    if (wide_weights) PTB_LMMA1(NFV, true); \
+    PTB_LMMA1(NFV, false);                 \
+  } while (0)
+  switch ((rank + 63) / 64) {
     case 1: PTB_LMMA(2);
     case 2: PTB_LMMA(4);
     case 3: PTB_LMMA(6);
@@ -666,14 +693,15 @@ PTB_API int ptb_latent_attention_mma(const float* q_abs, const void* q, int q_di
     case 7: PTB_LMMA(14);
     default: PTB_LMMA(16);
   }
+#undef PTB_LMMA1
 #undef PTB_LMMA
 }
 
 // ------------------------------------------------------------------------------------------------
-// Prompts in bfloat16 with per-head sizes that the tcgen05 prompt kernel takes (csrc/attention_tc.cu: 64 or
-// 128): the cached latents of the step's sequences are unfolded into per-head keys [W_uk[h] c | kr | 0] and
+// Prompts in bfloat16 with per-head sizes that the tcgen05 prompt kernel takes (csrc/attention_tc.cu: keys and
+// values of 64 or 128, or keys of 192 beside values of 128): the cached latents of the step's sequences are unfolded into per-head keys [W_uk[h] c | kr | 0] and
 // values [W_uv[h] c | 0] in scratch pools laid out like a cache entry's ([pages][heads][64][hd], the same
-// page numbers), and that kernel runs on them. The pieces here: the context's cache rows gathered into
+// page numbers; hd may differ between keys and values), and that kernel runs on them. The pieces here: the context's cache rows gathered into
 // dense matrices (for the library's product with [W_uk; W_uv]), the product's rows scattered into the
 // pools, the queries laid out as [plain | rotated | 0], and the output gate on the heads' first vdim entries.
 namespace {
@@ -693,7 +721,7 @@ __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ pool, Ste
 __global__ void latent_unfold_kernel(const __nv_bfloat16* __restrict__ kv, const __nv_bfloat16* __restrict__ kr_rows,
                                      StepBatch sb, const int* __restrict__ ctx_seq, const int* __restrict__ ctx_pos,
                                      __nv_bfloat16* __restrict__ k_tmp, __nv_bfloat16* __restrict__ v_tmp, int heads,
-                                     int dim, int rot_dim, int vdim, int hd) {
+                                     int dim, int rot_dim, int vdim, int hd, int hd_v) {
   const int i = blockIdx.x, seq = ctx_seq[i], pos = ctx_pos[i];
   const int page = sb.pages[size_t(seq) * sb.pages_stride + pos / PTB_PAGE], slot = pos % PTB_PAGE;
   const size_t width = size_t(heads) * (dim + vdim);
@@ -705,11 +733,11 @@ __global__ void latent_unfold_kernel(const __nv_bfloat16* __restrict__ kv, const
   }
   for (int idx = threadIdx.x; idx < heads * vdim; idx += blockDim.x) {
     const int h = idx / vdim, e = idx % vdim;
-    v_tmp[kv_offset(page, h, slot, heads, hd) + e] = row[size_t(heads) * dim + size_t(h) * vdim + e];
+    v_tmp[kv_offset(page, h, slot, heads, hd_v) + e] = row[size_t(heads) * dim + size_t(h) * vdim + e];
   }
 }
 
-__global__ void latent_q_unfold_kernel(const __nv_bfloat16* __restrict__ q, const float* __restrict__ rope_cos,
+__global__ void latent_q_unfold_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, const float* __restrict__ rope_cos,
                                        const float* __restrict__ rope_sin, int rot_pairs, int interleaved,
                                        __nv_bfloat16* __restrict__ out, int heads, int dim, int rot_dim, int hd) {
   const size_t t = blockIdx.x;
@@ -718,7 +746,7 @@ __global__ void latent_q_unfold_kernel(const __nv_bfloat16* __restrict__ q, cons
   for (int idx = threadIdx.x; idx < heads * items; idx += blockDim.x) {
     const int h = idx / items;
     int e = idx % items;
-    const __nv_bfloat16* src = q + (t * heads + h) * dq;
+    const __nv_bfloat16* src = q + t * q_stride + size_t(h) * dq;
     __nv_bfloat16* dst = out + (t * heads + h) * hd;
     if (e < dim) { dst[e] = src[e]; continue; }
     e -= dim;
@@ -737,15 +765,15 @@ __global__ void latent_q_unfold_kernel(const __nv_bfloat16* __restrict__ q, cons
   }
 }
 
-// out[t, h, :vdim] = o[t, h, :vdim] * sigmoid(gate[t, h, :vdim]); o rows are hd wide
+// out[t, h, :vdim] = o[t, h, :vdim] * sigmoid(gate[t, h, :vdim]), or * sigmoid(gate[t, h]) with per_head; o rows are hd wide
 __global__ void gate_heads_kernel(const __nv_bfloat16* __restrict__ o, const __nv_bfloat16* __restrict__ gate,
                                   long long gate_t, __nv_bfloat16* __restrict__ out, long long total, int heads, int vdim,
-                                  int hd) {
+                                  int hd, int per_head) {
   const size_t stride = size_t(gridDim.x) * blockDim.x;
   for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < size_t(total); i += stride) {
     const int e = int(i % vdim), h = int((i / vdim) % heads);
     const size_t t = i / (size_t(vdim) * heads);
-    const float g = to_f(gate[t * gate_t + size_t(h) * vdim + e]);
+    const float g = to_f(gate[t * gate_t + (per_head ? size_t(h) : size_t(h) * vdim + e)]);
     out[i] = __float2bfloat16_rn(to_f(o[(t * heads + h) * hd + e]) / (1.f + expf(-g)));
   }
 }
@@ -763,32 +791,32 @@ PTB_API int ptb_latent_gather(const void* pool, const StepBatch* sb, const int* 
 
 PTB_API int ptb_latent_unfold(const void* kv, const void* kr_rows, const StepBatch* sb, const int* ctx_seq,
                               const int* ctx_pos, int n_ctx, void* k_tmp, void* v_tmp, int heads, int dim, int rot_dim,
-                              int vdim, int hd, cudaStream_t stream) {
+                              int vdim, int hd, int hd_v, cudaStream_t stream) {
   if (n_ctx <= 0) return PTB_OK;
-  if (heads <= 0 || dim <= 0 || rot_dim < 0 || vdim <= 0 || dim + rot_dim > hd || vdim > hd) return PTB_ERR_SIZE;
+  if (heads <= 0 || dim <= 0 || rot_dim < 0 || vdim <= 0 || dim + rot_dim > hd || vdim > hd_v) return PTB_ERR_SIZE;
   latent_unfold_kernel<<<n_ctx, 256, 0, stream>>>((const __nv_bfloat16*)kv, (const __nv_bfloat16*)kr_rows, *sb, ctx_seq,
                                                   ctx_pos, (__nv_bfloat16*)k_tmp, (__nv_bfloat16*)v_tmp, heads, dim, rot_dim,
-                                                  vdim, hd);
+                                                  vdim, hd, hd_v);
   return launch_status();
 }
 
-PTB_API int ptb_latent_q_unfold(const void* q, const float* rope_cos, const float* rope_sin, int rot_pairs,
+PTB_API int ptb_latent_q_unfold(const void* q, long long q_stride, const float* rope_cos, const float* rope_sin, int rot_pairs,
                                 int interleaved, void* out, int n_tokens, int heads, int dim, int rot_dim, int hd,
                                 cudaStream_t stream) {
   if (n_tokens <= 0) return PTB_OK;
   if (heads <= 0 || dim <= 0 || rot_dim < 0 || dim + rot_dim > hd || 2 * rot_pairs > rot_dim) return PTB_ERR_SIZE;
   if (rot_pairs > 0 && (rope_cos == nullptr || rope_sin == nullptr)) return PTB_ERR_SIZE;
-  latent_q_unfold_kernel<<<n_tokens, 256, 0, stream>>>((const __nv_bfloat16*)q, rope_cos, rope_sin, rot_pairs, interleaved,
+  latent_q_unfold_kernel<<<n_tokens, 256, 0, stream>>>((const __nv_bfloat16*)q, q_stride, rope_cos, rope_sin, rot_pairs, interleaved,
                                                        (__nv_bfloat16*)out, heads, dim, rot_dim, hd);
   return launch_status();
 }
 
 PTB_API int ptb_gate_heads(const void* o, const void* gate, long long gate_t, void* out, int n_tokens, int heads, int vdim,
-                           int hd, cudaStream_t stream) {
+                           int hd, int per_head, cudaStream_t stream) {
   const long long total = (long long)n_tokens * heads * vdim;
   if (total <= 0) return PTB_OK;
   const size_t want = (size_t(total) + 255) / 256, most = size_t(sm_count()) * 16;
   gate_heads_kernel<<<int(want < most ? want : most), 256, 0, stream>>>((const __nv_bfloat16*)o, (const __nv_bfloat16*)gate,
-                                                                       gate_t, (__nv_bfloat16*)out, total, heads, vdim, hd);
+                                                                       gate_t, (__nv_bfloat16*)out, total, heads, vdim, hd, per_head);
   return launch_status();
 }

@@ -165,7 +165,8 @@ int launch_rglru_chunks(const float* gates, const void* u, const void* y_act, co
   return launch_status();
 }
 
-// y[t, g, :] = act(W[g] x[t, g, :] + bias[g]) [* sigmoid(gate[t, g, :])], W [groups, N, K]; x is read with
+// y[t, g, :] = act(W[g] x[t, g, :] + bias[g]) [* sigmoid(gate[t, g, :])], W [groups, N, K]; the gate's entry for
+// (t, g, n) lies at t gate_t + g gate_g + n gate_n (gate_n 0: one number per group); x is read with
 // strides (a token's stride xt, a group's stride xg), y [tokens, groups, N] is float32 or the input's
 // type. float32 FMAs in ascending k, 16 products summed apart and then into the total: a row's
 // result does not depend on the other rows of the launch. act: 0 none, 1 sigmoid.
@@ -175,7 +176,7 @@ template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 block_linear_kernel(const T* __restrict__ x, long long xt, long long xg, const T* __restrict__ w,
                     const float* __restrict__ bias, TO* __restrict__ y, const T* __restrict__ gate, long long gate_t,
-                    int M, int G, int N, int K, int act) {
+                    int gate_g, int gate_n, int M, int G, int N, int K, int act) {
   __shared__ float xs[BK][BM + 4];
   __shared__ float ws[BK][BN + 4];
   const int tid = threadIdx.x, g = blockIdx.z;
@@ -231,7 +232,7 @@ block_linear_kernel(const T* __restrict__ x, long long xt, long long xg, const T
       float v = acc[i][j];
       if (bias) v += bias[size_t(g) * N + gn];
       if (act == 1) v = 1.f / (1.f + expf(-v));
-      if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(gm) * gate_t + size_t(g) * N + gn])));
+      if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(gm) * gate_t + size_t(g) * gate_g + size_t(gn) * gate_n])));
       y[(size_t(gm) * G + g) * N + gn] = from_f<TO>(v);
     }
   }
@@ -260,7 +261,7 @@ template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
 block_linear_skinny_kernel(const T* __restrict__ x, long long xt, long long xg, const T* __restrict__ w,
                            const float* __restrict__ bias, TO* __restrict__ y, const T* __restrict__ gate,
-                           long long gate_t, int M, int G, int N, int K, int act, int vec) {
+                           long long gate_t, int gate_g, int gate_n, int M, int G, int N, int K, int act, int vec) {
   const int lane = threadIdx.x % 32;
   const long long item = (long long)blockIdx.x * (blockDim.x / 32) + threadIdx.x / 32;
   if (item >= (long long)G * N) return;
@@ -298,7 +299,7 @@ block_linear_skinny_kernel(const T* __restrict__ x, long long xt, long long xg, 
     if (lane == 0) {
       if (bias) v += bias[size_t(g) * N + n];
       if (act == 1) v = 1.f / (1.f + expf(-v));
-      if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(m) * gate_t + size_t(g) * N + n])));
+      if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(m) * gate_t + size_t(g) * gate_g + size_t(n) * gate_n])));
       y[(size_t(m) * G + g) * N + n] = from_f<TO>(v);
     }
   }
@@ -308,14 +309,14 @@ block_linear_skinny_kernel(const T* __restrict__ x, long long xt, long long xg, 
 // (float32 or bfloat16) -> y [M, groups, N] = act(z + bias[g]) [* sigmoid(gate)], float32 sums.
 template <typename TI, typename TO, typename TG>
 __global__ void block_epilogue_kernel(const TI* __restrict__ z, const float* __restrict__ bias, const TG* __restrict__ gate,
-                                      long long gate_t, TO* __restrict__ y, int M, int G, int N, int act) {
+                                      long long gate_t, int gate_g, int gate_n, TO* __restrict__ y, int M, int G, int N, int act) {
   const size_t total = size_t(M) * G * N, stride = size_t(gridDim.x) * blockDim.x;
   for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < total; i += stride) {
     const int n = int(i % N), g = int((i / N) % G), m = int(i / (size_t(N) * G));
     float v = to_f(z[(size_t(g) * M + m) * N + n]);
     if (bias) v += bias[size_t(g) * N + n];
     if (act == 1) v = 1.f / (1.f + expf(-v));
-    if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(m) * gate_t + size_t(g) * N + n])));
+    if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(m) * gate_t + size_t(g) * gate_g + size_t(n) * gate_n])));
     y[i] = from_f<TO>(v);
   }
 }
@@ -323,20 +324,21 @@ __global__ void block_epilogue_kernel(const TI* __restrict__ z, const float* __r
 }  // namespace
 
 PTB_API int ptb_block_epilogue(int in_dtype, int out_dtype, const void* z, const float* bias, const void* gate,
-                               long long gate_t, void* y, int M, int G, int N, int act, cudaStream_t stream) {
+                               long long gate_t, int gate_g, int gate_n, void* y, int M, int G, int N, int act,
+                               cudaStream_t stream) {
   if (M <= 0 || G <= 0 || N <= 0) return PTB_OK;
   if (act < 0 || act > 1) return PTB_ERR_SIZE;
   const size_t total = size_t(M) * G * N, want = (total + 255) / 256, most = size_t(sm_count()) * 16;
   const int blocks = int(want < most ? want : most);
   typedef __nv_bfloat16 bf;
   if (in_dtype == PTB_F32 && out_dtype == PTB_F32)
-    block_epilogue_kernel<float, float, bf><<<blocks, 256, 0, stream>>>((const float*)z, bias, (const bf*)gate, gate_t, (float*)y, M, G, N, act);
+    block_epilogue_kernel<float, float, bf><<<blocks, 256, 0, stream>>>((const float*)z, bias, (const bf*)gate, gate_t, gate_g, gate_n, (float*)y, M, G, N, act);
   else if (in_dtype == PTB_F32 && out_dtype == PTB_BF16)
-    block_epilogue_kernel<float, bf, bf><<<blocks, 256, 0, stream>>>((const float*)z, bias, (const bf*)gate, gate_t, (bf*)y, M, G, N, act);
+    block_epilogue_kernel<float, bf, bf><<<blocks, 256, 0, stream>>>((const float*)z, bias, (const bf*)gate, gate_t, gate_g, gate_n, (bf*)y, M, G, N, act);
   else if (in_dtype == PTB_BF16 && out_dtype == PTB_BF16)
-    block_epilogue_kernel<bf, bf, bf><<<blocks, 256, 0, stream>>>((const bf*)z, bias, (const bf*)gate, gate_t, (bf*)y, M, G, N, act);
+    block_epilogue_kernel<bf, bf, bf><<<blocks, 256, 0, stream>>>((const bf*)z, bias, (const bf*)gate, gate_t, gate_g, gate_n, (bf*)y, M, G, N, act);
   else if (in_dtype == PTB_BF16 && out_dtype == PTB_F32)
-    block_epilogue_kernel<bf, float, bf><<<blocks, 256, 0, stream>>>((const bf*)z, bias, (const bf*)gate, gate_t, (float*)y, M, G, N, act);
+    block_epilogue_kernel<bf, float, bf><<<blocks, 256, 0, stream>>>((const bf*)z, bias, (const bf*)gate, gate_t, gate_g, gate_n, (float*)y, M, G, N, act);
   else
     return PTB_ERR_DTYPE;
   return launch_status();
@@ -406,7 +408,8 @@ PTB_API int ptb_rglru_scan_chunks(int dtype, const float* gates, const void* u, 
 }
 
 PTB_API int ptb_block_linear(int dtype, int out_dtype, const void* x, long long xt, long long xg, const void* w,
-                             const float* bias, void* y, const void* gate, long long gate_t, int M, int G, int N,
+                             const float* bias, void* y, const void* gate, long long gate_t, int gate_g,
+                             int gate_n, int M, int G, int N,
                              int K, int act, cudaStream_t stream) {
   if (M <= 0 || G <= 0 || N <= 0) return PTB_OK;
   if (K <= 0 || act < 0 || act > 1 || G > 65535) return PTB_ERR_SIZE;
@@ -418,26 +421,26 @@ PTB_API int ptb_block_linear(int dtype, int out_dtype, const void* x, long long 
     typedef __nv_bfloat16 bf;
     const int vec = (K % 8 == 0 && xt % 8 == 0 && xg % 8 == 0 && aligned16(x) && aligned16(w)) ? 1 : 0;
     if (dtype == PTB_F32 && out_dtype == PTB_F32)
-      block_linear_skinny_kernel<float, float><<<sgrid, 256, 0, stream>>>((const float*)x, xt, xg, (const float*)w, bias, (float*)y, (const float*)gate, gate_t, M, G, N, K, act, vec);
+      block_linear_skinny_kernel<float, float><<<sgrid, 256, 0, stream>>>((const float*)x, xt, xg, (const float*)w, bias, (float*)y, (const float*)gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec);
     else if (dtype == PTB_BF16 && out_dtype == PTB_F32)
-      block_linear_skinny_kernel<bf, float><<<sgrid, 256, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (float*)y, (const bf*)gate, gate_t, M, G, N, K, act, vec);
+      block_linear_skinny_kernel<bf, float><<<sgrid, 256, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (float*)y, (const bf*)gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec);
     else if (dtype == PTB_BF16 && out_dtype == PTB_BF16)
-      block_linear_skinny_kernel<bf, bf><<<sgrid, 256, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (bf*)y, (const bf*)gate, gate_t, M, G, N, K, act, vec);
+      block_linear_skinny_kernel<bf, bf><<<sgrid, 256, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (bf*)y, (const bf*)gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec);
     else
       return PTB_ERR_DTYPE;
     return launch_status();
   }
   if (dtype == PTB_F32 && out_dtype == PTB_F32)
     block_linear_kernel<float, float><<<grid, 256, 0, stream>>>((const float*)x, xt, xg, (const float*)w, bias,
-                                                                (float*)y, (const float*)gate, gate_t, M, G, N, K, act);
+                                                                (float*)y, (const float*)gate, gate_t, gate_g, gate_n, M, G, N, K, act);
   else if (dtype == PTB_BF16 && out_dtype == PTB_F32)
     block_linear_kernel<__nv_bfloat16, float><<<grid, 256, 0, stream>>>(
         (const __nv_bfloat16*)x, xt, xg, (const __nv_bfloat16*)w, bias, (float*)y, (const __nv_bfloat16*)gate, gate_t,
-        M, G, N, K, act);
+        gate_g, gate_n, M, G, N, K, act);
   else if (dtype == PTB_BF16 && out_dtype == PTB_BF16)
     block_linear_kernel<__nv_bfloat16, __nv_bfloat16><<<grid, 256, 0, stream>>>(
         (const __nv_bfloat16*)x, xt, xg, (const __nv_bfloat16*)w, bias, (__nv_bfloat16*)y, (const __nv_bfloat16*)gate,
-        gate_t, M, G, N, K, act);
+        gate_t, gate_g, gate_n, M, G, N, K, act);
   else
     return PTB_ERR_DTYPE;
   return launch_status();

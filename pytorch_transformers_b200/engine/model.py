@@ -410,6 +410,11 @@ class CausalLM:
             rows, _ = self.final_norm.forward_pending(k.gather_rows(ctx.dev["logits_at"], x.base, self.status),
                                                       k.gather_rows(ctx.dev["logits_at"], x.pending, self.status), x.bias)
             return self.logits(rows)
+        if isinstance(x, DeferredSum) and x.bias is None and hasattr(self.final_norm, "forward_sum"):
+            x.join(x.base.device)       # likewise: the last sum at the wanted rows, in the final norm's kernel
+            rows = self.final_norm.forward_sum(k.gather_rows(ctx.dev["logits_at"], x.base, self.status),
+                                               k.gather_rows(ctx.dev["logits_at"], x.pending, self.status))[1]
+            return self.logits(rows)
         x = resolve(k, x)
         rows = k.gather_rows(ctx.dev["logits_at"], x, self.status)
         rows = self.final_norm.forward(rows)

@@ -75,6 +75,12 @@ def _check_rows(t: torch.Tensor, shape, dtype, what: str) -> None:
                           f"{tuple(t.shape)} of {t.dtype}, strides {t.stride()}")
 
 
+def _check_heads(q: torch.Tensor, what: str) -> None:
+    """``q`` is a CUDA tensor [tokens, heads, entries] whose heads lie side by side (tokens may lie wider apart)."""
+    if not q.is_cuda or q.dim() != 3 or q.stride(2) != 1 or (q.shape[1] > 1 and q.stride(1) != q.shape[2]):
+        raise KernelError(f"{what}: queries must be a CUDA tensor [tokens, heads, entries] with a token's heads side by side")
+
+
 _configured = False
 
 
@@ -104,7 +110,7 @@ def lib():
                      "ptb_mlstm_chunk_tokens", "ptb_embed_rows", "ptb_attention_generic_capped", "ptb_attention_mma_capped",
                      "ptb_qk_prepare_store", "ptb_route_grouped", "ptb_expert_combine_shared", "ptb_glu_act",
                      "ptb_head_norm_gate_act", "ptb_gla_decay", "ptb_gla_walk", "ptb_gla_chunks", "ptb_gla_max_dim",
-                     "ptb_gla_chunk_tokens"):
+                     "ptb_gla_chunk_tokens", "ptb_route_biased", "ptb_attention_tc_sizes", "ptb_attention_tc_supports_sizes"):
             getattr(L, name).restype = ctypes.c_int
         L.ptb_latent_part_floats.restype = ctypes.c_longlong
         L.ptb_expert_plan_words.restype = ctypes.c_longlong
@@ -520,26 +526,30 @@ def selftest_bounded_wait(device, tries: int = 1000) -> torch.Tensor:
     return gave_up
 
 
-def attention_tc_supports(head_dim: int) -> bool:
-    return bool(lib().ptb_attention_tc_supports(int(head_dim)))
+def attention_tc_supports(head_dim: int, v_dim: Optional[int] = None) -> bool:
+    return bool(lib().ptb_attention_tc_supports_sizes(int(head_dim), int(head_dim if v_dim is None else v_dim)))
 
 
 def attention_tc(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor, batch: StepBatchC,
                  tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tiles: int, kv_heads: int, scale: float,
-                 slopes: Optional[torch.Tensor] = None):
+                 slopes: Optional[torch.Tensor] = None, wide_weights: bool = False):
     """Causal prompt attention on tcgen05 tensor cores with accumulators in tensor memory: bfloat16,
-    head size 64 or 128, tiles of 128 tokens, no window; ``slopes`` [heads] float32: per-head score
-    slopes (ALiBi). Returns [tokens, heads * head_dim]."""
+    head size 64 or 128 (or keys of 192 entries beside values of 128), tiles of 128 tokens, no window; ``slopes``
+    [heads] float32: per-head score slopes (ALiBi). ``wide_weights``: the softmax weights meet the values as two
+    bfloat16 terms (16 bits of mantissa) instead of one; not with slopes. Returns [tokens, heads * v_dim]."""
     _need_cuda(q, k_pool, v_pool, tile_seq, tile_q0, slopes)
     if q.dtype != torch.bfloat16:
         raise KernelError("attention_tc takes bfloat16 tensors")
     n, heads, head_dim = q.shape
-    out = torch.empty((n, heads * head_dim), dtype=q.dtype, device=q.device)
-    if not k_pool.is_contiguous() or not v_pool.is_contiguous() or k_pool.shape != v_pool.shape:
+    v_dim = v_pool.shape[-1]
+    out = torch.empty((n, heads * v_dim), dtype=q.dtype, device=q.device)
+    if (not k_pool.is_contiguous() or not v_pool.is_contiguous() or k_pool.shape[:-1] != v_pool.shape[:-1]
+            or k_pool.shape[-1] != head_dim):
         raise KernelError("attention_tc takes the contiguous K and V pools of one cache entry")
-    _check(lib().ptb_attention_tc(_ptr(q), _ptr(k_pool), _ptr(v_pool), k_pool.shape[0], _ptr(out), ctypes.byref(batch), _ptr(tile_seq),
-                                  _ptr(tile_q0), n_tiles, _ptr(slopes), heads, kv_heads, head_dim, ctypes.c_float(scale),
-                                  _ptr(error_flag(q.device)), _stream(q)), "attention_tc")
+    _check(lib().ptb_attention_tc_sizes(_ptr(q), _ptr(k_pool), _ptr(v_pool), k_pool.shape[0], _ptr(out), ctypes.byref(batch),
+                                        _ptr(tile_seq), _ptr(tile_q0), n_tiles, _ptr(slopes), heads, kv_heads, head_dim, v_dim,
+                                        ctypes.c_float(scale), 1 if wide_weights else 0, _ptr(error_flag(q.device)),
+                                        _stream(q)), "attention_tc")
     return out
 
 
@@ -836,14 +846,16 @@ def latent_attention_mma_supports(rank: int, rot_dim: int) -> bool:
 def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, q_rot_off: int, pool: torch.Tensor, batch: StepBatchC,
                      tile_seq: torch.Tensor, tile_q0: torch.Tensor, n_tiles: int, tile_tokens: int, rope, rank: int,
                      rot_dim: int, scale: float, interleaved: bool = True, n_splits: int = 1,
-                     tensor_cores: Optional[bool] = None) -> torch.Tensor:
+                     tensor_cores: Optional[bool] = None, wide_weights: bool = False) -> torch.Tensor:
     """Causal attention in latent space. ``q_abs`` [tokens, heads, rank] float32 (queries with the key
-    up-projection folded in), ``q`` [tokens, heads, q_dim] whose entries from ``q_rot_off`` on are the part
-    to rotate, ``pool`` the cache entry's rows [pages, 1, 64, rank + rot_dim]. A tile holds ``tile_tokens``
-    tokens x 16 / tile_tokens heads; ``n_splits`` blocks share a tile's key pages. bfloat16 with ``rank`` a
-    multiple of 64 and ``rot_dim`` of 16 runs on the tensor cores (``tensor_cores=False``: the general kernel). Returns
+    up-projection folded in), ``q`` [tokens, heads, q_dim] (a view whose tokens may lie wider apart) whose entries from
+    ``q_rot_off`` on are the part to rotate, ``pool`` the cache entry's rows [pages, 1, 64, rank + rot_dim]. A tile holds ``tile_tokens``
+    tokens x 16 / tile_tokens heads; ``n_splits`` blocks share a tile's key pages. bfloat16 with ``rank`` and
+    ``rot_dim`` multiples of 16 runs on the tensor cores (``tensor_cores=False``: the general kernel), with
+    ``wide_weights`` with the softmax weights as two bfloat16 terms. Returns
     [tokens, heads, rank] in the model dtype: per head, the softmax-weighted sum of the cached latents."""
-    _need_cuda(q_abs, q, pool, tile_seq, tile_q0)
+    _need_cuda(q_abs, pool, tile_seq, tile_q0)
+    _check_heads(q, "latent_attention")
     n, heads, q_dim = q.shape
     if q_abs.dtype != torch.float32 or tuple(q_abs.shape) != (n, heads, rank) or pool.dtype != q.dtype:
         raise KernelError("latent_attention: q_abs must be float32 [tokens, heads, rank] and the pool of q's dtype")
@@ -863,13 +875,13 @@ def latent_attention(q_abs: torch.Tensor, q: torch.Tensor, q_rot_off: int, pool:
         need = int(lib().ptb_latent_part_floats(n_tiles, heads, heads_per_block, n_splits, rank))
         part = torch.empty(need, dtype=torch.float32, device=q.device)
     if tensor_cores:
-        _check(lib().ptb_latent_attention_mma(_ptr(q_abs), _ptr(q), q_dim, q_rot_off, _ptr(pool), _ptr(part), _ptr(out),
+        _check(lib().ptb_latent_attention_mma(_ptr(q_abs), _ptr(q), ctypes.c_longlong(q.stride(0)), q_dim, q_rot_off, _ptr(pool), _ptr(part), _ptr(out),
                                               ctypes.byref(batch), _ptr(tile_seq), _ptr(tile_q0), n_tiles, _ptr(cos),
                                               _ptr(sin), pairs, 1 if interleaved else 0, heads, rank, rot_dim, tile_tokens,
-                                              heads_per_block, ctypes.c_float(scale), n_splits, _stream(q)),
+                                              heads_per_block, ctypes.c_float(scale), n_splits, 1 if wide_weights else 0, _stream(q)),
                "latent_attention_mma")
     else:
-        _check(lib().ptb_latent_attention(_dtype_code(q), _ptr(q_abs), _ptr(q), q_dim, q_rot_off, _ptr(pool), _ptr(part),
+        _check(lib().ptb_latent_attention(_dtype_code(q), _ptr(q_abs), _ptr(q), ctypes.c_longlong(q.stride(0)), q_dim, q_rot_off, _ptr(pool), _ptr(part),
                                           _ptr(out), ctypes.byref(batch), _ptr(tile_seq), _ptr(tile_q0), n_tiles, _ptr(cos),
                                           _ptr(sin), pairs, 1 if interleaved else 0, heads, rank, rot_dim, tile_tokens,
                                           heads_per_block, ctypes.c_float(scale), n_splits, _stream(q)), "latent_attention")
@@ -883,15 +895,20 @@ def latent_unfolded_attention(q: torch.Tensor, pool: torch.Tensor, k_tmp: torch.
                               w_ukv: torch.Tensor, gate: torch.Tensor, batch: StepBatchC, ctx_seq: torch.Tensor,
                               ctx_pos: torch.Tensor, n_ctx: int, mtile_seq: torch.Tensor, mtile_q0: torch.Tensor,
                               n_mma_tiles: int, rope, dim: int, rot_dim: int, vdim: int, rank: int, scale: float,
-                              interleaved: bool = True) -> torch.Tensor:
+                              interleaved: bool = True, gate_per_head: bool = False,
+                              wide_weights: bool = False) -> torch.Tensor:
     """Latent attention of prompts through the tcgen05 prompt kernel (bfloat16): the ``n_ctx`` cached rows
     (``ctx_seq``, ``ctx_pos``: sequence and position of each) of the step's sequences are unfolded with
     ``w_ukv`` = [W_uk; W_uv] into per-head keys and values in the scratch pools ``k_tmp`` / ``v_tmp``
-    ([pages, heads, 64, hd], zero outside what is written here), the queries are laid out to match, and
-    ``attention_tc`` runs on them. Returns the heads' outputs times sigmoid(gate): [tokens, heads * vdim]."""
-    _need_cuda(q, pool, k_tmp, v_tmp, w_ukv, ctx_seq, ctx_pos)
+    ([pages, heads, 64, hd], zero outside what is written here; hd may differ between the two), the queries (a view
+    whose tokens may lie wider apart) are laid out to match, and ``attention_tc`` runs on them. Returns the heads'
+    outputs times sigmoid(gate): [tokens, heads * vdim]; ``gate`` [tokens, heads * vdim], or [tokens, heads] with
+    ``gate_per_head``. ``wide_weights``: as attention_tc takes it."""
+    _need_cuda(pool, k_tmp, v_tmp, w_ukv, ctx_seq, ctx_pos)
+    _check_heads(q, "latent_unfolded_attention")
     n, heads, dq = q.shape
-    hd = k_tmp.shape[-1]
+    hd, hd_v = k_tmp.shape[-1], v_tmp.shape[-1]
+    _check_rows(gate, (n, heads if gate_per_head else heads * vdim), q.dtype, "latent_unfolded_attention: gate")
     if q.dtype != torch.bfloat16 or dq != dim + rot_dim or tuple(w_ukv.shape) != (heads * (dim + vdim), rank):
         raise KernelError("latent_unfolded_attention: sizes or dtypes do not fit")
     cos, sin = rope if rope is not None else (None, None)
@@ -903,14 +920,14 @@ def latent_unfolded_attention(q: torch.Tensor, pool: torch.Tensor, k_tmp: torch.
                                    _ptr(kr_rows), rank, rot_dim, stream), "latent_gather")
     kv = matmul_nt(c_rows, w_ukv)
     _check(lib().ptb_latent_unfold(_ptr(kv), _ptr(kr_rows), ctypes.byref(batch), _ptr(ctx_seq), _ptr(ctx_pos), n_ctx,
-                                   _ptr(k_tmp), _ptr(v_tmp), heads, dim, rot_dim, vdim, hd, stream), "latent_unfold")
+                                   _ptr(k_tmp), _ptr(v_tmp), heads, dim, rot_dim, vdim, hd, hd_v, stream), "latent_unfold")
     q_tc = torch.empty((n, heads, hd), dtype=q.dtype, device=q.device)
-    _check(lib().ptb_latent_q_unfold(_ptr(q), _ptr(cos), _ptr(sin), pairs, 1 if interleaved else 0, _ptr(q_tc), n, heads,
+    _check(lib().ptb_latent_q_unfold(_ptr(q), ctypes.c_longlong(q.stride(0)), _ptr(cos), _ptr(sin), pairs, 1 if interleaved else 0, _ptr(q_tc), n, heads,
                                      dim, rot_dim, hd, stream), "latent_q_unfold")
-    o = attention_tc(q_tc, k_tmp, v_tmp, batch, mtile_seq, mtile_q0, n_mma_tiles, heads, scale)
+    o = attention_tc(q_tc, k_tmp, v_tmp, batch, mtile_seq, mtile_q0, n_mma_tiles, heads, scale, wide_weights=wide_weights)
     out = torch.empty((n, heads * vdim), dtype=q.dtype, device=q.device)
-    _check(lib().ptb_gate_heads(_ptr(o), _ptr(gate), ctypes.c_longlong(gate.stride(0)), _ptr(out), n, heads, vdim, hd,
-                                stream), "gate_heads")
+    _check(lib().ptb_gate_heads(_ptr(o), _ptr(gate), ctypes.c_longlong(gate.stride(0)), _ptr(out), n, heads, vdim, hd_v,
+                                1 if gate_per_head else 0, stream), "gate_heads")
     return out
 
 
@@ -920,18 +937,21 @@ BLOCK_LINEAR_LIBRARY_ROWS = 256   # rows from which block_linear's product is th
 
 
 def block_linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, act: str = "none",
-                 out_dtype: Optional[torch.dtype] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                 out_dtype: Optional[torch.dtype] = None, gate: Optional[torch.Tensor] = None,
+                 gate_per_group: bool = False) -> torch.Tensor:
     """y[t, g] = act(w[g] @ x[t, g] + bias[g]) [* sigmoid(gate[t, g])]: ``x`` [tokens, groups, K] (any
     strides with unit stride along K), ``w`` [groups, N, K], ``bias`` [groups, N] float32, ``gate``
-    [tokens, groups * N] (rows may be wider apart). ``act``: "none" or "sigmoid". Returns
+    [tokens, groups * N] (rows may be wider apart), or with ``gate_per_group`` [tokens, groups], a number per group. ``act``: "none" or "sigmoid". Returns
     [tokens, groups, N] in ``out_dtype`` (float32, or the input's dtype)."""
     _need_cuda(w, bias)
     m, g, k = x.shape
     n = w.shape[1]
     if x.stride(2) != 1 or tuple(w.shape) != (g, n, k) or w.dtype != x.dtype:
         raise KernelError("block_linear: shapes or dtypes do not fit")
-    if gate is not None and (gate.stride(1) != 1 or tuple(gate.shape) != (m, g * n) or gate.dtype != x.dtype):
-        raise KernelError("block_linear: the gate does not fit")
+    gate_at = (0, 0, 0)       # strides of the gate along tokens, groups and a group's outputs
+    if gate is not None:
+        _check_rows(gate, (m, g if gate_per_group else g * n), x.dtype, "block_linear: gate")
+        gate_at = (gate.stride(0),) + ((1, 0) if gate_per_group else (n, 1))
     out_dtype = out_dtype or x.dtype
     y = torch.empty((m, g, n), dtype=out_dtype, device=x.device)
     if x.dtype == torch.bfloat16 and m >= BLOCK_LINEAR_LIBRARY_ROWS:
@@ -942,12 +962,12 @@ def block_linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] 
         else:
             z = torch.bmm(x.transpose(0, 1), w.transpose(1, 2))
         _check(lib().ptb_block_epilogue(_dtype_code(z), _dtype_code(y), _ptr(z), _ptr(bias), _ptr(gate),
-                                        ctypes.c_longlong(0 if gate is None else gate.stride(0)), _ptr(y), m, g, n,
+                                        ctypes.c_longlong(gate_at[0]), gate_at[1], gate_at[2], _ptr(y), m, g, n,
                                         {"none": 0, "sigmoid": 1}[act], _stream(x)), "block_epilogue")
         return y
     _check(lib().ptb_block_linear(_dtype_code(x), _dtype_code(y), _ptr(x), ctypes.c_longlong(x.stride(0)),
                                   ctypes.c_longlong(x.stride(1)), _ptr(w), _ptr(bias), _ptr(y), _ptr(gate),
-                                  ctypes.c_longlong(0 if gate is None else gate.stride(0)), m, g, n, k,
+                                  ctypes.c_longlong(gate_at[0]), gate_at[1], gate_at[2], m, g, n, k,
                                   {"none": 0, "sigmoid": 1}[act], _stream(x)), "block_linear")
     return y
 
@@ -1016,11 +1036,12 @@ EXPERT_TILE_ROWS = (16, 64)   # rows of a tile of the grouped products: few pair
 EXPERT_MMA_TILE_ROWS = (64, 128)   # rows of a tile of the tensor-core kernel
 
 
-ROUTE_SCORES = {"softmax": 0, "sigmoid": 1}
+ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "softmax_chosen": 2}
 
 
 def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Tensor], n_groups: int, keep: int, top: int,
-          scale: float, score: str = "softmax", extra: int = 0, group_top: int = 1, normalize: bool = False):
+          scale: float, score: str = "softmax", extra: int = 0, group_top: int = 1, normalize: bool = False,
+          bias: Optional[torch.Tensor] = None):
     """Router of a mixture of experts, float32: scores = softmax over all outputs (or a sigmoid per output),
     choice by score + correction (None: no correction) among the ``keep`` best of ``n_groups`` groups,
     weights = score * scale. Returns (ids int32 [tokens, top], weights float32 [tokens, top]).
@@ -1028,19 +1049,23 @@ def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Te
     ``group_top`` 2: a group is scored by the sum of its two largest choice scores instead of its largest.
     ``normalize``: weights = score / (sum of the chosen scores + 1e-20) * scale. ``extra``: the last ``extra`` rows of
     ``w_router`` are no router outputs; their logits are formed with the others (same input, same float32 sums) and the
-    call returns (ids, weights, logits float32 [tokens, outputs + extra])."""
-    _need_cuda(h, w_router, correction)
+    call returns (ids, weights, logits float32 [tokens, outputs + extra]). ``bias`` (float32 [outputs]) is part of the
+    logits. ``score`` "softmax_chosen": the choice is by the logits (+ correction), the weights are the softmax over the
+    chosen logits alone, times scale."""
+    _need_cuda(h, w_router, correction, bias)
     n_tokens, width = h.shape
     n = w_router.shape[0] - int(extra)
     if (w_router.dtype != torch.float32 or (correction is not None and correction.dtype != torch.float32)
             or w_router.shape[1] != width):
         raise KernelError("route: the router's matrix and correction are float32 [outputs, width] and [outputs]")
+    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != n):
+        raise KernelError("route: the logits' bias is float32 [outputs]")
     ids = torch.empty((n_tokens, top), dtype=torch.int32, device=h.device)
     gates = torch.empty((n_tokens, top), dtype=torch.float32, device=h.device)
     logits = torch.empty((n_tokens, n + int(extra)), dtype=torch.float32, device=h.device)
-    _check(lib().ptb_route_grouped(_dtype_code(h), _ptr(h), _ptr(w_router), _ptr(correction), _ptr(logits), _ptr(ids),
-                                   _ptr(gates), n_tokens, width, n, n_groups, keep, top, ctypes.c_float(scale),
-                                   ROUTE_SCORES[score], int(extra), int(group_top), 1 if normalize else 0, _stream(h)),
+    _check(lib().ptb_route_biased(_dtype_code(h), _ptr(h), _ptr(w_router), _ptr(bias), _ptr(correction), _ptr(logits),
+                                  _ptr(ids), _ptr(gates), n_tokens, width, n, n_groups, keep, top, ctypes.c_float(scale),
+                                  ROUTE_SCORES[score], int(extra), int(group_top), 1 if normalize else 0, _stream(h)),
            "route")
     global launches
     launches += 1       # the logits and the choice are two kernels
@@ -1050,14 +1075,15 @@ def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Te
 def routed_experts(h: torch.Tensor, ids: torch.Tensor, gates: torch.Tensor, w_gate_up: torch.Tensor,
                    w_down: torch.Tensor, base: Optional[torch.Tensor] = None, mma_tile_rows: int = 0,
                    plain_act: Optional[str] = None, shared: Optional[torch.Tensor] = None,
-                   shared_gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   shared_gate: Optional[torch.Tensor] = None, weigh_output: bool = False) -> torch.Tensor:
     """base + sum over a token's choices of weight * expert(h): experts ``w_gate_up`` [E, 2 F, width]
     (gate rows, then up rows) and ``w_down`` [E, width, F] compute down(silu(gate h) * (up h)); an id >= E
     is an identity expert. Pairs are sorted by expert on the device and run as tiles of grouped
     products. Returns [tokens, width] in ``base``'s dtype (float32 without a base).
 
     With ``plain_act`` (an activation's name) the experts have no gate and take their weight on the input:
-    ``w_gate_up`` is [E, F, width] and the result is base + sum of down(act(up (weight * h))).
+    ``w_gate_up`` is [E, F, width] and the result is base + sum of down(act(up (weight * h))); with ``weigh_output``
+    they too take it on the output, base + sum of weight * down(act(up h)).
 
     ``shared`` (float32 [tokens, width]): the result of an expert that every token uses, added in the same kernel, times
     sigmoid(``shared_gate``) where that is given (float32 [tokens, 1], a view whose rows may lie wider apart)."""
@@ -1071,7 +1097,8 @@ def routed_experts(h: torch.Tensor, ids: torch.Tensor, gates: torch.Tensor, w_ga
     n_experts, two_f, _ = w_gate_up.shape
     f = two_f // 2 if plain_act is None else two_f
     first, act = (0, 0) if plain_act is None else (2, ACTIVATIONS[plain_act])
-    scale = None if plain_act is None else gates
+    on_input = plain_act is not None and not weigh_output
+    scale = gates if on_input else None
     pairs = n_tokens * top
     # bfloat16 with row sizes in whole 16-byte words: the tensor-core kernel (tiles of 64 rows); else float32 FMAs
     mma = h.dtype == torch.bfloat16 and width % 8 == 0 and f % 8 == 0
@@ -1106,7 +1133,7 @@ def routed_experts(h: torch.Tensor, ids: torch.Tensor, gates: torch.Tensor, w_ga
     out = torch.empty((n_tokens, width), dtype=torch.float32 if base is None else base.dtype, device=h.device)
     row_of_pair = plan[1 + 3 * max_tiles:1 + 3 * max_tiles + pairs]
     _check(L.ptb_expert_combine_shared(code, _dtype_code(out), _ptr(base), _ptr(h), _ptr(y), _ptr(ids),
-                                       _ptr(gates if plain_act is None else None),
+                                       _ptr(None if on_input else gates),
                                        _ptr(row_of_pair), _ptr(out), n_tokens, width, top, _ptr(shared), _ptr(shared_gate),
                                        0 if shared_gate is None else shared_gate.stride(0), stream), "expert_combine")
     return out

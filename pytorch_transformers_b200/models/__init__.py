@@ -10,6 +10,8 @@ from ..config.pogezen import PogezenConfig
 from .pogezen import pogezen_spec
 from ..config.figudra import FigudraConfig
 from .figudra import figudra_spec
+from ..config.vesidra import VesidraConfig
+from .vesidra import vesidra_spec
 
 register_architecture(
     "falcon", ("FalconForCausalLM", "RWForCausalLM"), FalconConfig, falcon_spec, name_rules=FALCON_NAME_RULES,
@@ -19,3 +21,4 @@ register_architecture("pafevik", ("Pafevik",), PafevikConfig, pafevik_spec)
 register_architecture("zalunex", ("Zalunex",), ZalunexConfig, zalunex_spec)
 register_architecture("pogezen", ("Pogezen",), PogezenConfig, pogezen_spec)
 register_architecture("figudra", ("Figudra",), FigudraConfig, figudra_spec)
+register_architecture("vesidra", ("Vesidra",), VesidraConfig, vesidra_spec)

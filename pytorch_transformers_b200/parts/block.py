@@ -13,6 +13,8 @@ Sums are formed in float32 and rounded once; where the model keeps its residual 
 """
 from __future__ import annotations
 
+import torch
+
 from .base import BuildContext, DeferredSum, NormedStream, Part, PartSpec, register_part, resolve
 
 
@@ -60,6 +62,12 @@ class ParallelBlock(Part):
                 m = a
         if two_streams:
             return self._forward_two_streams(x, a, m, ctx, entry, side)
+        if (self.feed_forward is not None and getattr(self.feed_forward, "adds_in_sum", False)
+                and getattr(self.mixer, "wide_out", False) and x.dtype == torch.float32):
+            # a feed-forward whose last kernel is a sum takes the float32 stream as one more term of it; the mixer's float32
+            # sums stay pending, as the feed-forward's do below
+            mixed = self.mixer.forward(a, ctx, entry)
+            return DeferredSum(self.feed_forward.forward(m, ctx, add=x), mixed)
         mixed = _plus(k, self.mixer, x, a, ctx, entry)           # x + mixer
         if self.feed_forward is None:
             return mixed
@@ -77,7 +85,6 @@ class ParallelBlock(Part):
         parallel branches per block. The mixer's launches come first: with the feed-forward's first,
         its blocks take the SMs and the mixer's short kernels queue behind them (15 % slower).
         Tensors that cross streams stay referenced until the step ends."""
-        import torch
         main = torch.cuda.current_stream(x.device)
         side.wait_stream(main)
         with torch.cuda.stream(side):
@@ -102,7 +109,6 @@ class SequentialBlock(Part):
     def _defers(self, x) -> bool:
         """Elementwise norms on a float32 stream, under a mixer and a feed-forward that can leave their last sum to the
         next norm's kernel: no sum of this block is a kernel of its own."""
-        import torch
         fuses = getattr(self.mixer, "fuses_norm", None)
         base = x.base if isinstance(x, DeferredSum) else x
         return (fuses is not None and fuses(self.norm_mixer) and getattr(self.mixer, "defers_sums", lambda: False)()
@@ -163,7 +169,6 @@ class SandwichBlock(Part):
                 raise ValueError("the sandwich block's norms are RMS norms without bias")
 
     def forward(self, x, ctx, entry):
-        import torch
         k = self.build.kernels
         opened = x.normed if isinstance(x, NormedStream) and x.by is self.norm_mixer else None
         x = resolve(k, x)

@@ -10,8 +10,10 @@ stream in float32 in the same kernel.
 
 Variants, all by constructor parameters: ``score="sigmoid"`` scores every output by a sigmoid of its own
 instead of the softmax; ``correction=False`` has no correction tensor; ``expert="plain"`` experts have no
-gate, ``W_down act(W_up h)`` with ``activation`` by name; ``weight_on="input"`` multiplies the expert's
-input by the weight instead of its output: the result is the sum of ``expert(weight * h)``.
+gate, ``W_down act(W_up h)`` with ``activation`` by name; ``weight_on="input"`` (plain experts only) multiplies the
+expert's input by the weight instead of its output: the result is the sum of ``expert(weight * h)``.
+``router_bias=True``: the logits are ``W_r h + b``. ``score="softmax_chosen"``: the choice is by the logits (+ correction)
+and the weights are the softmax over the chosen logits alone, times ``scale``.
 ``group_score="top2_sum"`` scores a group by the sum of its two largest choice scores instead of its largest.
 ``normalize=True`` divides the chosen outputs' scores by their sum (+ 1e-20) before ``scale``. A ``shared`` child (a
 feed-forward part that returns float32 sums) is an expert that every token uses; its result is added in the kernel
@@ -31,11 +33,13 @@ from .base import BuildContext, ParamDecl, Part, PartSpec, register_part
 class RoutedExperts(Part):
     graph_safe = True
     fuses_add = True
+    adds_in_sum = True      # a tensor to add is one more term of the last kernel's sum
 
     def __init__(self, build: BuildContext, spec: PartSpec, hidden: int, inner: int, experts: int, top: int,
                  identity: int = 0, groups: int = 1, keep: int = 1, scale: float = 1.0, score: str = "softmax",
                  correction: bool = True, expert: str = "gated_silu", activation: str = "gelu",
-                 weight_on: str = "output", group_score: str = "max", normalize: bool = False, shared_gate: bool = False):
+                 weight_on: str = "output", group_score: str = "max", normalize: bool = False, shared_gate: bool = False,
+                 router_bias: bool = False):
         super().__init__(build, spec)
         if group_score not in ("max", "top2_sum"):
             raise ValueError(f"a group's score is 'max' or 'top2_sum', got {group_score!r}")
@@ -48,11 +52,14 @@ class RoutedExperts(Part):
             raise ValueError(f"router scores are one of {', '.join(build.kernels.ROUTE_SCORES)}, got {score!r}")
         if expert not in ("gated_silu", "plain") or weight_on not in ("output", "input"):
             raise ValueError(f"experts are 'gated_silu' or 'plain' and weigh their 'output' or 'input', got {expert!r}, {weight_on!r}")
-        if (expert == "plain") != (weight_on == "input"):
+        if expert != "plain" and weight_on == "input":
             # the grouped kernels take the weight in the plain expert's first epilogue, or in the sum of outputs
-            raise ValueError("plain experts weigh their input and gated experts their output")
+            raise ValueError("gated experts weigh their output")
         if expert == "plain" and (activation not in build.kernels.ACTIVATIONS or identity):
             raise ValueError(f"plain experts take an activation of {', '.join(build.kernels.ACTIVATIONS)} and no identity experts")
+        self.weight_on, self.has_router_bias = weight_on, bool(router_bias)
+        if normalize and score == "softmax_chosen":
+            raise ValueError("the softmax over the chosen logits is normalised already")
         self.score, self.has_correction, self.expert, self.activation = score, bool(correction), expert, activation
         self.hidden, self.inner, self.experts, self.top = int(hidden), int(inner), int(experts), int(top)
         self.identity, self.groups, self.keep, self.scale = int(identity), int(groups), int(keep), float(scale)
@@ -63,13 +70,15 @@ class RoutedExperts(Part):
             raise ValueError(f"cannot choose {self.top} of {n} outputs in {self.keep} of {self.groups} groups")
         if n > 512:
             raise ValueError(f"the router kernel takes up to 512 outputs, got {n}")
-        self.p_router = self.p_correction = self.p_gate_up = self.p_down = None
+        self.p_router = self.p_router_b = self.p_correction = self.p_gate_up = self.p_down = None
 
     def param_decls(self) -> Dict[str, ParamDecl]:
         n = self.experts + self.identity
         d = {"router": ParamDecl((n, self.hidden), role="vector")}
         if self.has_correction:
             d["correction"] = ParamDecl((n,), role="vector")
+        if self.has_router_bias:
+            d["router_b"] = ParamDecl((n,), role="vector")
         if self.has_shared_gate:
             d["shared_gate"] = ParamDecl((1, self.hidden), role="vector")
         for e in range(self.experts):
@@ -81,6 +90,7 @@ class RoutedExperts(Part):
 
     def bind(self, t: Dict[str, torch.Tensor]) -> None:
         self.p_router, self.p_correction = t["router"].contiguous(), t.get("correction")
+        self.p_router_b = t.get("router_b")
         if self.has_shared_gate:        # one more row of the router's product: the shared expert's gate
             self.p_router = torch.cat([self.p_router, t["shared_gate"].reshape(1, self.hidden)]).contiguous()
         E, F = self.experts, self.inner
@@ -103,7 +113,7 @@ class RoutedExperts(Part):
             add = add()
         routed = k.route(x, self.p_router, self.p_correction, self.groups, self.keep, self.top, self.scale, self.score,
                          extra=1 if self.has_shared_gate else 0, group_top=2 if self.group_score == "top2_sum" else 1,
-                         normalize=self.normalize)
+                         normalize=self.normalize, bias=self.p_router_b)
         ids, weights = routed[0], routed[1]
         shared = shared_gate = None
         if self.shared is not None:
@@ -112,4 +122,4 @@ class RoutedExperts(Part):
                 shared_gate = routed[2][:, self.experts + self.identity:]
         return k.routed_experts(x, ids, weights, self.p_gate_up, self.p_down, base=add,
                                 plain_act=self.activation if self.expert == "plain" else None, shared=shared,
-                                shared_gate=shared_gate)
+                                shared_gate=shared_gate, weigh_output=self.weight_on == "output")

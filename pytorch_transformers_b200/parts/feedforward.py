@@ -14,12 +14,15 @@ from .linear import linear, linear_pending
 class DenseFeedForward(Part):
     graph_safe = True
     def __init__(self, build: BuildContext, spec: PartSpec, hidden: int, inner: int, activation: str = "gelu",
-                 bias: bool = False):
+                 bias: bool = False, wide_out: bool = False):
         super().__init__(build, spec)
         if activation not in build.kernels.ACTIVATIONS:
             raise ValueError(f"activation {activation!r} is not supported "
                              f"(supported: {', '.join(build.kernels.ACTIVATIONS)})")
         self.hidden, self.inner, self.activation, self.has_bias = int(hidden), int(inner), activation, bool(bias)
+        self.wide_out = bool(wide_out)      # without a tensor to add: the last product's float32 sums, unrounded
+        if self.wide_out and self.has_bias:
+            raise ValueError("a feed-forward with biases does not return its last product's bare sums")
         self.p_up_weight = self.p_up_bias = self.p_down_weight = self.p_down_bias = None
 
     def param_decls(self) -> Dict[str, ParamDecl]:
@@ -36,6 +39,8 @@ class DenseFeedForward(Part):
         u = linear(k, x, self.p_up_weight, self.p_up_bias, self.activation)
         if callable(add):
             add = add()   # resolved as late as possible: the caller may still be producing it on another stream
+        if add is None and self.wide_out:
+            return linear(k, u, self.p_down_weight, wide_out=True)
         return linear(k, u, self.p_down_weight, self.p_down_bias, add=add)
 
     def forward_pending(self, x, ctx):
