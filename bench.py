@@ -1068,7 +1068,108 @@ def run_figudra(args):
     return 0
 
 
+# ---- Vesidra beside Pafevik at equal size (`--only vesidra [--size s|m]`) ----
+# Sizes that resemble a served model's layers: the width; four parallel layers of latent attention with 16 or 32 heads of
+# 96 plain + 32 rotated query/key entries (YaRN frequencies) and values of 128, a key/value latent of 512 and a gate per
+# head; layers 0 and 2 over a gated unit 4 x the width wide, layers 1 and 3 over 64 plain experts of 1,408 of which a token
+# uses 6 and a shared expert of 2,816. Pafevik beside it has four layers of latent attention of the same heads, sizes and
+# latent (queries through a latent of their own, a gate per entry) over 64 gated experts of 1,408 of which a token uses 6.
+# `vesidra_192` is Vesidra with heads of 128 plain + 64 rotated entries.
+def vesidra_config(size, dim=96, rot_dim=32):
+    z = PAFEVIK_SIZES[size]
+    w, heads = z["width"], z["heads"]
+    att = {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": 128, "kv_rank": 512, "scale": (dim + rot_dim) ** -0.5,
+           "rot": {"base": 10000.0, "dims": rot_dim, "scaling": {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    glu = {"kind": "dense", "ff": 4 * w}
+    moe = {"kind": "moe", "expert": {"ff": 1408}, "shared": {"ff": 2816}, "router": {"experts": 64, "top": 6}}
+    return {"architecture": "Vesidra", "vocab": 32000, "width": w, "embedding": {"scale": w ** 0.5}, "norm": {"eps": 1e-6},
+            "layers": [{"type": "latent_attention", "mixer": dict(att), "mlp": f} for f in (glu, moe, glu, moe)]}
+
+
+def pafevik_attention_config(size):
+    raw = pafevik_config(size)
+    raw["layers"] = [dict(raw["layers"][0], mixer=dict(raw["layers"][0]["mixer"])) for _ in range(4)]
+    return raw
+
+
+def run_vesidra(args):
+    import torch
+
+    import pytorch_transformers_b200 as ptb
+
+    torch.cuda.set_device(0)
+    pk = peaks()
+    gen = torch.Generator().manual_seed(0)
+    tokens, batch, context = args.prefill_tokens, args.batch, args.context
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    raws = {"vesidra": vesidra_config(args.size), "vesidra_192": vesidra_config(args.size, 128, 64),
+            "pafevik": pafevik_attention_config(args.size)}
+    w = raws["vesidra"]["width"]
+    result = {"only": "vesidra", "size": args.size, "prefill_tokens": tokens, "batch": batch, "context": context,
+              "config": {"width": w, "layers": 4, "heads": raws["vesidra"]["layers"][0]["mixer"]["heads"]}}
+    for name, raw in raws.items():
+        cls = ptb.PafevikConfig if name == "pafevik" else ptb.VesidraConfig
+        model = ptb.AutoModelForCausalLM.from_config(cls.from_dict(raw), seed=0, dtype="bfloat16")
+        result[name] = measure_prefill_and_decode(model, args, gen, flush)
+        del model
+        torch.cuda.empty_cache()
+
+    roof = {}
+    pairs, scored = tokens * 6, tokens * (tokens + 1) // 2
+
+    def put(name, value, peak, unit):
+        roof[f"{name}_{unit}"] = round(value, 1)
+        roof[f"{name}_frac_of_{'hbm' if unit == 'GBps' else 'burst'}"] = round(value / peak, 4)
+
+    for name, raw in raws.items():
+        table, m = result[name]["prefill_kernels_ms"], raw["layers"][0]["mixer"]
+        H, dq, vd, rank = m["heads"], m["dim"] + m["rot_dim"], m["vdim"], m["kv_rank"]
+
+        def per_call(key):
+            return table[key]["ms"] / table[key]["calls"] if key in table else None
+
+        for key in ("latent_attention", "latent_unfolded_attention"):
+            t = per_call(key)
+            if t:   # scores and outputs over the visible pairs; the unfolded form also its up-projection
+                flops = H * scored * 2 * ((dq + vd) if key != "latent_attention" else (2 * rank + m["rot_dim"]))
+                put(f"{name}_{key}", (flops + (2 * tokens * rank * H * (m["dim"] + vd) if key != "latent_attention" else 0)) / t / 1e9,
+                    pk["bf16_tflops"], "TFLOPs")
+        t = per_call("attention_tc")
+        if t:       # the tcgen05 kernel of the unfolded form alone
+            put(f"{name}_attention_tc", H * scored * 2 * (dq + vd) / t / 1e9, pk["bf16_tflops"], "TFLOPs")
+        t = per_call("routed_experts")
+        if t:
+            put(f"{name}_experts", pairs * (3 if name == "pafevik" else 2) * 2 * w * 1408 / t / 1e9, pk["bf16_tflops"], "TFLOPs")
+        t = per_call("route")
+        if t:
+            roof[f"{name}_route_us"] = round(t * 1e3, 1)
+        t = per_call("norm_stream")
+        if t:       # Vesidra's norms also form the stream's last sum
+            put(f"{name}_norm_stream", tokens * w * ((4 + 4 + 4 + 2) if name != "pafevik" else (4 + 2)) / t / 1e6, pk["hbm_gbs"], "GBps")
+        t = per_call("add_stream")
+        if t:
+            put(f"{name}_add_stream", tokens * w * 12 / t / 1e6, pk["hbm_gbs"], "GBps")
+        t = per_call("glu_act")
+        if t:
+            put(f"{name}_glu_act", tokens * 4 * w * 6 / t / 1e6, pk["hbm_gbs"], "GBps")
+        t = table.get("matmul_nt")
+        if t:       # all library products of the prompt but the head's (one row)
+            if name == "pafevik":
+                q = m["q_rank"] * (w + H * dq)
+                flops = 2 * tokens * 4 * (q + w * (rank + m["rot_dim"] + H * vd) + w * H * vd + rank * H * (m["dim"] + vd))
+            else:
+                flops = 2 * tokens * (4 * (w * (H * dq + rank + m["rot_dim"] + H) + w * H * vd + rank * H * (m["dim"] + vd))
+                                      + 2 * 3 * w * 4 * w + 2 * 2 * w * 2816)
+            put(f"{name}_library_products", flops / t["ms"] / 1e9, pk["bf16_tflops"], "TFLOPs")
+    result["roofline"] = roof
+    result["peaks"] = pk
+    print(json.dumps(result))
+    return 0
+
+
 def run_ours(args):
+    if args.only == "vesidra":
+        return run_vesidra(args)
     if args.only == "figudra":
         return run_figudra(args)
     if args.only == "pafevik":
@@ -1352,10 +1453,10 @@ def main():
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration's (0: all)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "sample", "decode-attention", "prefill-attention", "config", "linear",
-                             "fill", "mma-cadence", "pafevik", "zalunex", "pogezen", "figudra"],
+                             "fill", "mma-cadence", "pafevik", "zalunex", "pogezen", "figudra", "vesidra"],
                     help="run one section only and print its numbers (for profilers)")
     ap.add_argument("--shape", default="7b", choices=sorted(SHAPES), help="model shape for --only decode / prefill")
-    ap.add_argument("--size", default="s", choices=sorted(PAFEVIK_SIZES), help="layer sizes for --only pafevik, --only zalunex, --only pogezen and --only figudra")
+    ap.add_argument("--size", default="s", choices=sorted(PAFEVIK_SIZES), help="layer sizes for --only pafevik, --only zalunex, --only pogezen, --only figudra and --only vesidra")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="prompt length for --only prefill")
     ap.add_argument("--context", type=int, default=CONTEXT, help="cached tokens per sequence for --only decode")
     ap.add_argument("--past", type=int, default=0, help="cached tokens before the prompt for --only prefill-attention")

@@ -17,34 +17,75 @@ constexpr int ROUTE_VPL = 16;   // router outputs per lane: up to 512 outputs
 constexpr int ROUTE_WARPS = 8;
 
 constexpr int ROUTE_TOKENS = 8;   // tokens of a block of the logits kernel for prompts: a matrix row is read once for them
+constexpr int ROUTE_OUTPUTS = 2;  // outputs of a warp there: a token's row is read once for them
 
-// Router logits z[t, e] = W_r[e] . h[t] in float32: a warp per output, lanes along the width, TPB tokens a
-// block; a token's sums have one fixed order whatever else is in the batch.
-template <typename T, int TPB>
+__device__ __forceinline__ void load4(const float* p, float (&f)[4]) {
+  const float4 v = *reinterpret_cast<const float4*>(p);
+  f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+}
+__device__ __forceinline__ void load4(const __nv_bfloat16* p, float (&f)[4]) {
+  const uint2 v = *reinterpret_cast<const uint2*>(p);
+  f[0] = __uint_as_float(v.x << 16); f[1] = __uint_as_float(v.x & 0xffff0000u);
+  f[2] = __uint_as_float(v.y << 16); f[3] = __uint_as_float(v.y & 0xffff0000u);
+}
+
+// Router logits z[t, e] = W_r[e] . h[t] + bias[e] in float32: EPW outputs a warp, lanes along the width, TPB tokens a
+// block; a token's sums have one fixed order whatever else is in the batch. VEC: a lane takes four neighbouring k at a time
+// (the host checks: the width a multiple of 4, rows at whole words); the order then depends on the width alone.
+template <typename T, int TPB, int EPW, bool VEC>
 __global__ void __launch_bounds__(32 * ROUTE_WARPS)
 route_logits_kernel(const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ bias,
                     float* __restrict__ z, int n_tokens, int width, int n, int n_bias) {
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
-  const int t0 = blockIdx.x * TPB, e = blockIdx.y * ROUTE_WARPS + warp;
-  if (e >= n) return;
-  const float* wr = w_router + size_t(e) * width;
-  float d[TPB];
+  const int t0 = blockIdx.x * TPB, e0 = (blockIdx.y * ROUTE_WARPS + warp) * EPW;
+  if (e0 >= n) return;
+  float d[EPW][TPB];
   const T* rows[TPB];      // a token past the end reads the block's first token; its result is not written
+  const float* wr[EPW];    // likewise an output past the end
+#pragma unroll
+  for (int j = 0; j < EPW; ++j) wr[j] = w_router + size_t(e0 + j < n ? e0 + j : e0) * width;
 #pragma unroll
   for (int i = 0; i < TPB; ++i) {
-    d[i] = 0.f;
     rows[i] = h + size_t(t0 + i < n_tokens ? t0 + i : t0) * width;
+#pragma unroll
+    for (int j = 0; j < EPW; ++j) d[j][i] = 0.f;
   }
+  if (VEC) {
+#pragma unroll 2
+    for (int k = lane * 4; k < width; k += 128) {
+      float wv[EPW][4];
+#pragma unroll
+      for (int j = 0; j < EPW; ++j) load4(wr[j] + k, wv[j]);
+#pragma unroll
+      for (int i = 0; i < TPB; ++i) {
+        float hv[4];
+        load4(rows[i] + k, hv);
+#pragma unroll
+        for (int j = 0; j < EPW; ++j)
+#pragma unroll
+          for (int u = 0; u < 4; ++u) d[j][i] = fmaf(wv[j][u], hv[u], d[j][i]);
+      }
+    }
+  } else {
 #pragma unroll 4
-  for (int k = lane; k < width; k += 32) {
-    const float wv = wr[k];
+    for (int k = lane; k < width; k += 32) {
 #pragma unroll
-    for (int i = 0; i < TPB; ++i) d[i] = fmaf(wv, to_f(rows[i][k]), d[i]);
+      for (int j = 0; j < EPW; ++j) {
+        const float wv = wr[j][k];
+#pragma unroll
+        for (int i = 0; i < TPB; ++i) d[j][i] = fmaf(wv, to_f(rows[i][k]), d[j][i]);
+      }
+    }
   }
 #pragma unroll
-  for (int i = 0; i < TPB; ++i) {
-    const float v = warp_sum(d[i]) + (bias != nullptr && e < n_bias ? bias[e] : 0.f);
-    if (lane == 0 && t0 + i < n_tokens) z[size_t(t0 + i) * n + e] = v;
+  for (int j = 0; j < EPW; ++j) {
+    const int e = e0 + j;
+    const float b = bias != nullptr && e < n_bias ? bias[e] : 0.f;
+#pragma unroll
+    for (int i = 0; i < TPB; ++i) {
+      const float v = warp_sum(d[j][i]) + b;
+      if (lane == 0 && e < n && t0 + i < n_tokens) z[size_t(t0 + i) * n + e] = v;
+    }
   }
 }
 
@@ -375,19 +416,24 @@ PTB_API int ptb_route_biased(int dtype, const void* h, const float* w_router, co
       top > (n / n_groups) * keep || width <= 0 || score_kind < 0 || score_kind > 2 || extra < 0 || group_top < 1 || group_top > 2)
     return PTB_ERR_SIZE;
   // few tokens (steps of single tokens): one token a block, so that the blocks fill the device
-  const int tpb = n_tokens >= 2 * sm_count() ? ROUTE_TOKENS : 1;
-  dim3 grid((n_tokens + tpb - 1) / tpb, (n + extra + ROUTE_WARPS - 1) / ROUTE_WARPS);
-#define PTB_ROUTE(TT, NTOK) \
-  route_logits_kernel<TT, NTOK><<<grid, 32 * ROUTE_WARPS, 0, stream>>>((const TT*)h, w_router, bias, logits, n_tokens, width, n + extra, n)
-  if (dtype == PTB_F32) {
-    if (tpb == 1) PTB_ROUTE(float, 1);
-    else PTB_ROUTE(float, ROUTE_TOKENS);
-  } else if (dtype == PTB_BF16) {
-    if (tpb == 1) PTB_ROUTE(__nv_bfloat16, 1);
-    else PTB_ROUTE(__nv_bfloat16, ROUTE_TOKENS);
-  } else {
-    return PTB_ERR_DTYPE;
-  }
+  const bool many = n_tokens >= 2 * sm_count();
+  const int tpb = many ? ROUTE_TOKENS : 1, epw = many ? ROUTE_OUTPUTS : 1;
+  dim3 grid((n_tokens + tpb - 1) / tpb, (n + extra + ROUTE_WARPS * epw - 1) / (ROUTE_WARPS * epw));
+  const bool vec = width % 4 == 0 && aligned16(h) && aligned16(w_router);
+#define PTB_ROUTE2(TT, NTOK, NOUT, V)                                                                               \
+  route_logits_kernel<TT, NTOK, NOUT, V><<<grid, 32 * ROUTE_WARPS, 0, stream>>>((const TT*)h, w_router, bias, logits, \
+                                                                                n_tokens, width, n + extra, n)
+#define PTB_ROUTE(TT)                                              \
+  do {                                                             \
+    if (many && vec) PTB_ROUTE2(TT, ROUTE_TOKENS, ROUTE_OUTPUTS, true);  \
+    else if (many) PTB_ROUTE2(TT, ROUTE_TOKENS, ROUTE_OUTPUTS, false);   \
+    else if (vec) PTB_ROUTE2(TT, 1, 1, true);                      \
+    else PTB_ROUTE2(TT, 1, 1, false);                              \
+  } while (0)
+  if (dtype == PTB_F32) PTB_ROUTE(float);
+  else if (dtype == PTB_BF16) PTB_ROUTE(__nv_bfloat16);
+  else return PTB_ERR_DTYPE;
+#undef PTB_ROUTE2
 #undef PTB_ROUTE
   if (launch_status() != PTB_OK) return PTB_ERR_LAUNCH;
   const size_t smem = size_t(ROUTE_WARPS) * (n + n_groups) * sizeof(float);

@@ -15,6 +15,10 @@ namespace {
 constexpr int ROWS = 16;      // (token, head) rows of a tile
 constexpr int THREADS = 128;  // 8 threads per row
 
+// A row of a split's partial result: `rank` unnormalised sums, the running maximum, the sum of the weights; rows start
+// at whole 16-byte words.
+__host__ __device__ __forceinline__ int part_row(int rank) { return (rank + 2 + 3) / 4 * 4; }
+
 // One block per token: the row `src` [rank + rot_dim] of the down-projection becomes the cached row:
 // the first `rank` entries divided by their root mean square (eps inside the root) times norm_w,
 // the last rot_dim rotated by the token's position (pairs (2i, 2i+1) when interleaved, else
@@ -199,16 +203,15 @@ latent_attention_kernel(const float* __restrict__ q_abs, const T* __restrict__ q
     }
   }
   if (n_splits > 1) {
-    float* p = part + ((size_t(tile) * gridDim.y + blockIdx.y) * n_splits + split) * ROWS * size_t(rank + 2) +
-               size_t(r) * (rank + 2);
+    float* p = part + (((size_t(tile) * gridDim.y + blockIdx.y) * n_splits + split) * ROWS + r) * part_row(rank);
     if (c == 0) {
-      p[0] = m_run;
-      p[1] = l_run;
+      p[rank] = m_run;
+      p[rank + 1] = l_run;
     }
 #pragma unroll
     for (int i = 0; i < DPT; ++i) {
       const int e = c + 8 * i;
-      if (e < rank) p[2 + e] = acc[i];
+      if (e < rank) p[e] = acc[i];
     }
     return;
   }
@@ -223,39 +226,70 @@ latent_attention_kernel(const float* __restrict__ q_abs, const T* __restrict__ q
   }
 }
 
-// merges the splits of a tile in ascending order of their pages: one block per (tile, head chunk, row)
+// Merges the splits of a tile in ascending order of their pages: one block per (tile, head chunk, row). The first warp
+// turns the splits' maxima into their weights; then a thread takes four columns (one where rank is no multiple of 4) and has
+// eight splits' loads in flight.
 template <typename T>
-__global__ void latent_join_kernel(const float* __restrict__ part, T* __restrict__ out, StepBatch sb,
-                                   const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, int heads,
-                                   int rank, int tile_tokens, int heads_per_block, int n_splits) {
+__global__ void __launch_bounds__(128)
+latent_join_kernel(const float* __restrict__ part, T* __restrict__ out, StepBatch sb,
+                   const int* __restrict__ tile_seq, const int* __restrict__ tile_q0, int heads,
+                   int rank, int tile_tokens, int heads_per_block, int n_splits) {
   extern __shared__ float jw[];   // the splits' weights exp(m_s - m) / l
   const int tile = blockIdx.x, h0 = blockIdx.y * heads_per_block, r = blockIdx.z;
   const int seq = tile_seq[tile], q0 = tile_q0[tile];
   const int toks = min(tile_tokens, sb.seq_new[seq] - q0), start = sb.seq_start[seq];
   const int ti = r / heads_per_block, hh = h0 + r % heads_per_block;
   if (!(ti < toks && hh < heads && r < tile_tokens * heads_per_block)) return;
-  const float* base = part + (size_t(tile) * gridDim.y + blockIdx.y) * n_splits * ROWS * size_t(rank + 2) + size_t(r) * (rank + 2);
-  const size_t split_stride = size_t(ROWS) * (rank + 2);
+  const int row = part_row(rank);
+  const float* base = part + ((size_t(tile) * gridDim.y + blockIdx.y) * n_splits * ROWS + r) * row;
+  const size_t split_stride = size_t(ROWS) * row;
   if (threadIdx.x < 32) {
     float m = -INFINITY;
-    for (int s = threadIdx.x; s < n_splits; s += 32) m = fmaxf(m, base[s * split_stride]);
+    for (int s = threadIdx.x; s < n_splits; s += 32) m = fmaxf(m, base[s * split_stride + rank]);
     m = warp_max(m);
     float l = 0.f;
-    for (int s = 0; s < n_splits; ++s) {      // ascending order, the same in every lane
-      const float ms = base[s * split_stride];
+    for (int s = threadIdx.x; s < n_splits; s += 32) {
+      const float ms = base[s * split_stride + rank];
       const float w = (ms == -INFINITY) ? 0.f : expf(ms - m);
-      l += base[s * split_stride + 1] * w;
-      if (threadIdx.x == 0) jw[s] = w;
+      l += base[s * split_stride + rank + 1] * w;
+      jw[s] = w;
     }
-    __syncwarp();
+    l = warp_sum(l);
     const float inv = l > 0.f ? 1.f / l : 0.f;
     for (int s = threadIdx.x; s < n_splits; s += 32) jw[s] *= inv;
   }
   __syncthreads();
   T* o = out + (size_t(start + q0 + ti) * heads + hh) * rank;
+  constexpr int AHEAD = 8;
+  if (rank % 4 == 0) {
+    for (int e = threadIdx.x * 4; e < rank; e += blockDim.x * 4) {
+      float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int s0 = 0; s0 < n_splits; s0 += AHEAD) {
+        float4 x[AHEAD];
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u)
+          if (s0 + u < n_splits) x[u] = *reinterpret_cast<const float4*>(base + (s0 + u) * split_stride + e);
+#pragma unroll
+        for (int u = 0; u < AHEAD; ++u)
+          if (s0 + u < n_splits) {
+            const float w = jw[s0 + u];
+            v.x = fmaf(x[u].x, w, v.x);
+            v.y = fmaf(x[u].y, w, v.y);
+            v.z = fmaf(x[u].z, w, v.z);
+            v.w = fmaf(x[u].w, w, v.w);
+          }
+      }
+      o[e] = from_f<T>(v.x);
+      o[e + 1] = from_f<T>(v.y);
+      o[e + 2] = from_f<T>(v.z);
+      o[e + 3] = from_f<T>(v.w);
+    }
+    return;
+  }
   for (int e = threadIdx.x; e < rank; e += blockDim.x) {
     float v = 0.f;
-    for (int s = 0; s < n_splits; ++s) v = fmaf(base[s * split_stride + 2 + e], jw[s], v);
+#pragma unroll 8
+    for (int s = 0; s < n_splits; ++s) v = fmaf(base[s * split_stride + e], jw[s], v);
     o[e] = from_f<T>(v);
   }
 }
@@ -312,7 +346,7 @@ PTB_API int ptb_latent_rows() { return ROWS; }
 PTB_API long long ptb_latent_part_floats(int n_tiles, int heads, int heads_per_block, int n_splits, int rank) {
   if (n_splits <= 1) return 0;
   const long long chunks = (heads + heads_per_block - 1) / heads_per_block;
-  return (long long)n_tiles * chunks * n_splits * ROWS * (rank + 2);
+  return (long long)n_tiles * chunks * n_splits * ROWS * part_row(rank);
 }
 
 PTB_API int ptb_latent_store(int dtype, const void* src, long long src_stride, const float* norm_w, float eps,
@@ -409,13 +443,31 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
   float* wmax = wmax_all + tg * 64;
   float* wsum = wsum_all + tg * 64;
 
+  const int last_pos = past + q0 + toks - 1;
+  const int n_blocks = last_pos / PTB_PAGE + 1;
+  const int per = (n_blocks + n_splits - 1) / n_splits;
+  const int kb_lo = split * per, kb_hi = min(n_blocks, kb_lo + per) - 1;
+  const int* pages = sb.pages + size_t(seq) * sb.pages_stride;
+  const int chunks = dk / 8;
+  // a page's rows, a warp a row at a time
+  auto fetch = [&](int kb) {
+    const __nv_bfloat16* kp = pool + kv_offset(pages[kb], 0, 0, 1, dk);
+    const uint32_t dst = smem_u32(k_s);
+    for (int j = tid / 32; j < PTB_PAGE; j += NT / 32)
+      for (int c = lane; c < chunks; c += 32) cp_async16(dst + j * rowb + c * 16, kp + size_t(j) * dk + c * 8);
+    cp_async_commit();
+  };
+  if (kb_lo <= kb_hi) fetch(kb_lo);      // on its way while the query rows are formed
+
   // the query rows, rounded to bfloat16: [q_abs | rotated part]
-  for (int i = tid; i < QROWS * rank; i += NT) {
-    const int rr = i / rank, e = i % rank;
+  for (int rr = tid / 32; rr < QROWS; rr += NT / 32) {
     const int ti = rr / heads_per_block, hh = h0 + rr % heads_per_block;
     const bool ok = ti < toks && hh < heads && rr < used_rows;
-    const float v = ok ? q_abs[(size_t(start + q0 + ti) * heads + hh) * rank + e] : 0.f;
-    reinterpret_cast<__nv_bfloat16*>(q_s + rr * rowb)[e] = __float2bfloat16_rn(v);
+    const float* src = q_abs + (size_t(start + q0 + ti) * heads + hh) * rank;
+    for (int e = lane * 4; e < rank; e += 128) {
+      const float4 v = ok ? *reinterpret_cast<const float4*>(src + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+      *reinterpret_cast<uint2*>(q_s + rr * rowb + e * 2) = make_uint2(pack_bf16(v.x, v.y), pack_bf16(v.z, v.w));
+    }
   }
   const int items = rot_pairs + (rot_dim - 2 * rot_pairs);
   for (int i = tid; i < QROWS * items; i += NT) {
@@ -453,26 +505,17 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
     for (int c = 0; c < 4; ++c) acc[j][c] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
 
-  const int last_pos = past + q0 + toks - 1;
-  const int n_blocks = last_pos / PTB_PAGE + 1;
-  const int per = (n_blocks + n_splits - 1) / n_splits;
-  const int kb_lo = split * per, kb_hi = min(n_blocks, kb_lo + per) - 1;
-  const int* pages = sb.pages + size_t(seq) * sb.pages_stride;
-  const int chunks = dk / 8;
   const uint32_t q_base = smem_u32(q_s) + tg * 16 * rowb, k_base = smem_u32(k_s), p_base = smem_u32(p_s);
   const int col0 = warp * NF * 8;       // first output column of this warp
   const int my_pairs = min(NF / 2, max(0, rank - col0) / 16);   // groups of 16 columns that this warp has
 
   for (int kb = kb_lo; kb <= kb_hi; ++kb) {
-    const __nv_bfloat16* kp = pool + kv_offset(pages[kb], 0, 0, 1, dk);
-    __syncthreads();   // the page before is no longer read (and the query rows are written)
-    for (int i = tid; i < PTB_PAGE * chunks; i += NT) {
-      const int j = i / chunks, c = i % chunks;
-      cp_async16(k_base + j * rowb + c * 16, kp + size_t(j) * dk + c * 8);
+    if (kb > kb_lo) {
+      __syncthreads();   // the page before is no longer read
+      fetch(kb);
     }
-    cp_async_commit();
     cp_async_wait<0>();
-    __syncthreads();
+    __syncthreads();     // the page has landed for everybody (and the query rows are written)
     // scores of keys 16 warp .. 16 warp + 15
     float s[2][4];
 #pragma unroll
@@ -585,17 +628,15 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
   for (int hf = 0; hf < 2; ++hf) {
     const int rl = hf ? r_hi : r_lo, rr = tg * 16 + rl;
     if (n_splits > 1) {      // only with TG = 1
-      float* p = part + ((size_t(tile) * gridDim.y + blockIdx.y) * n_splits + split) * ROWS * size_t(rank + 2) +
-                 size_t(rl) * (rank + 2);
+      float* p = part + (((size_t(tile) * gridDim.y + blockIdx.y) * n_splits + split) * ROWS + rl) * part_row(rank);
       if (warp == 0 && lane % 4 == 0) {
-        p[0] = m_run[hf];
-        p[1] = l_run[hf];
+        p[rank] = m_run[hf];
+        p[rank + 1] = l_run[hf];
       }
 #pragma unroll
       for (int j = 0; j < NF; ++j) {
         if (j >= 2 * my_pairs) continue;
-        p[2 + col0 + j * 8 + c0] = acc[j][hf * 2];
-        p[2 + col0 + j * 8 + c0 + 1] = acc[j][hf * 2 + 1];
+        *reinterpret_cast<float2*>(p + col0 + j * 8 + c0) = make_float2(acc[j][hf * 2], acc[j][hf * 2 + 1]);
       }
     } else if (pos_of[hf] >= 0) {
       const int ti = rr / heads_per_block, hh = h0 + rr % heads_per_block;
@@ -673,7 +714,7 @@ PTB_API int ptb_latent_attention_mma(const float* q_abs, const void* q, long lon
     return PTB_ERR_SIZE;
   if (n_splits > 1 && part == nullptr) return PTB_ERR_SIZE;
   if (rot_pairs > 0 && (rope_cos == nullptr || rope_sin == nullptr)) return PTB_ERR_SIZE;
-  if (!aligned16(pool) || !aligned16(out)) return PTB_ERR_ALIGN;
+  if (!aligned16(pool) || !aligned16(out) || !aligned16(q_abs) || !aligned16(part)) return PTB_ERR_ALIGN;
 #define PTB_LMMA1(NFV, W)                                                                                              \
   return launch_latent_mma<NFV, W>(q_abs, q, q_stride, q_dim, q_rot_off, pool, part, out, *sb, tile_seq, tile_q0, n_tiles, \
                                    rope_cos, rope_sin, rot_pairs, interleaved, heads, rank, rot_dim, tile_tokens,        \
@@ -717,39 +758,54 @@ __global__ void latent_gather_kernel(const __nv_bfloat16* __restrict__ pool, Ste
   for (int e = threadIdx.x; e < rot_dim; e += blockDim.x) kr_rows[size_t(i) * rot_dim + e] = src[rank + e];
 }
 
+// V entries at a time: 8 (16-byte words) where every row and every part of a row is whole words, else 1
+template <int V> struct Word;
+template <> struct Word<1> { typedef __nv_bfloat16 type; };
+template <> struct Word<8> { typedef uint4 type; };
+
 // kv [ctx, heads * dim + heads * vdim]: a context row's keys of all heads, then its values of all heads
+template <int V>
 __global__ void latent_unfold_kernel(const __nv_bfloat16* __restrict__ kv, const __nv_bfloat16* __restrict__ kr_rows,
                                      StepBatch sb, const int* __restrict__ ctx_seq, const int* __restrict__ ctx_pos,
                                      __nv_bfloat16* __restrict__ k_tmp, __nv_bfloat16* __restrict__ v_tmp, int heads,
                                      int dim, int rot_dim, int vdim, int hd, int hd_v) {
+  typedef typename Word<V>::type W;
   const int i = blockIdx.x, seq = ctx_seq[i], pos = ctx_pos[i];
   const int page = sb.pages[size_t(seq) * sb.pages_stride + pos / PTB_PAGE], slot = pos % PTB_PAGE;
   const size_t width = size_t(heads) * (dim + vdim);
   const __nv_bfloat16* row = kv + size_t(i) * width;
-  const int dq = dim + rot_dim;
+  const int dq = (dim + rot_dim) / V, dv = vdim / V;
   for (int idx = threadIdx.x; idx < heads * dq; idx += blockDim.x) {
-    const int h = idx / dq, e = idx % dq;
-    k_tmp[kv_offset(page, h, slot, heads, hd) + e] = (e < dim) ? row[size_t(h) * dim + e] : kr_rows[size_t(i) * rot_dim + (e - dim)];
+    const int h = idx / dq, e = (idx % dq) * V;
+    *reinterpret_cast<W*>(k_tmp + kv_offset(page, h, slot, heads, hd) + e) =
+        *reinterpret_cast<const W*>((e < dim) ? row + size_t(h) * dim + e : kr_rows + size_t(i) * rot_dim + (e - dim));
   }
-  for (int idx = threadIdx.x; idx < heads * vdim; idx += blockDim.x) {
-    const int h = idx / vdim, e = idx % vdim;
-    v_tmp[kv_offset(page, h, slot, heads, hd_v) + e] = row[size_t(heads) * dim + size_t(h) * vdim + e];
+  for (int idx = threadIdx.x; idx < heads * dv; idx += blockDim.x) {
+    const int h = idx / dv, e = (idx % dv) * V;
+    *reinterpret_cast<W*>(v_tmp + kv_offset(page, h, slot, heads, hd_v) + e) =
+        *reinterpret_cast<const W*>(row + size_t(heads) * dim + size_t(h) * vdim + e);
   }
 }
 
+template <int V>
 __global__ void latent_q_unfold_kernel(const __nv_bfloat16* __restrict__ q, long long q_stride, const float* __restrict__ rope_cos,
                                        const float* __restrict__ rope_sin, int rot_pairs, int interleaved,
                                        __nv_bfloat16* __restrict__ out, int heads, int dim, int rot_dim, int hd) {
+  typedef typename Word<V>::type W;
   const size_t t = blockIdx.x;
   const int dq = dim + rot_dim;
-  const int items = dim + rot_pairs + (rot_dim - 2 * rot_pairs) + (hd - dq);     // per head: plain, pairs, unrotated rest, padding
+  // per head: plain words, pairs, unrotated rest, padding words
+  const int plain = dim / V, rest = rot_dim - 2 * rot_pairs, pad = (hd - dq) / V, items = plain + rot_pairs + rest + pad;
   for (int idx = threadIdx.x; idx < heads * items; idx += blockDim.x) {
     const int h = idx / items;
     int e = idx % items;
     const __nv_bfloat16* src = q + t * q_stride + size_t(h) * dq;
     __nv_bfloat16* dst = out + (t * heads + h) * hd;
-    if (e < dim) { dst[e] = src[e]; continue; }
-    e -= dim;
+    if (e < plain) {
+      *reinterpret_cast<W*>(dst + e * V) = *reinterpret_cast<const W*>(src + e * V);
+      continue;
+    }
+    e -= plain;
     if (e < rot_pairs) {
       const int ia = interleaved ? 2 * e : e, ib = interleaved ? 2 * e + 1 : e + rot_pairs;
       float a, b;
@@ -759,22 +815,32 @@ __global__ void latent_q_unfold_kernel(const __nv_bfloat16* __restrict__ q, long
       continue;
     }
     e -= rot_pairs;
-    if (e < rot_dim - 2 * rot_pairs) { dst[dim + 2 * rot_pairs + e] = src[dim + 2 * rot_pairs + e]; continue; }
-    e -= rot_dim - 2 * rot_pairs;
-    dst[dq + e] = __float2bfloat16_rn(0.f);
+    if (e < rest) { dst[dim + 2 * rot_pairs + e] = src[dim + 2 * rot_pairs + e]; continue; }
+    e -= rest;
+    *reinterpret_cast<W*>(dst + dq + e * V) = W{};
   }
 }
 
 // out[t, h, :vdim] = o[t, h, :vdim] * sigmoid(gate[t, h, :vdim]), or * sigmoid(gate[t, h]) with per_head; o rows are hd wide
+template <int V>
 __global__ void gate_heads_kernel(const __nv_bfloat16* __restrict__ o, const __nv_bfloat16* __restrict__ gate,
-                                  long long gate_t, __nv_bfloat16* __restrict__ out, long long total, int heads, int vdim,
+                                  long long gate_t, __nv_bfloat16* __restrict__ out, long long words, int heads, int vdim,
                                   int hd, int per_head) {
+  typedef typename Word<V>::type W;
   const size_t stride = size_t(gridDim.x) * blockDim.x;
-  for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < size_t(total); i += stride) {
-    const int e = int(i % vdim), h = int((i / vdim) % heads);
-    const size_t t = i / (size_t(vdim) * heads);
-    const float g = to_f(gate[t * gate_t + (per_head ? size_t(h) : size_t(h) * vdim + e)]);
-    out[i] = __float2bfloat16_rn(to_f(o[(t * heads + h) * hd + e]) / (1.f + expf(-g)));
+  const unsigned dv = unsigned(vdim / V);
+  for (size_t i = size_t(blockIdx.x) * blockDim.x + threadIdx.x; i < size_t(words); i += stride) {
+    const size_t th = i / dv;       // token * heads + head
+    const int e = int(i % dv) * V;
+    const size_t t = th / unsigned(heads);
+    const int h = int(th % unsigned(heads));
+    const __nv_bfloat16* g = gate + t * gate_t + (per_head ? size_t(h) : size_t(h) * vdim + e);
+    W w = *reinterpret_cast<const W*>(o + th * hd + e);
+    __nv_bfloat16* x = reinterpret_cast<__nv_bfloat16*>(&w);
+    const float one = 1.f + expf(-to_f(g[0]));
+#pragma unroll
+    for (int u = 0; u < V; ++u) x[u] = __float2bfloat16_rn(to_f(x[u]) / (per_head || u == 0 ? one : 1.f + expf(-to_f(g[u]))));
+    *reinterpret_cast<W*>(out + th * vdim + e) = w;
   }
 }
 
@@ -794,9 +860,15 @@ PTB_API int ptb_latent_unfold(const void* kv, const void* kr_rows, const StepBat
                               int vdim, int hd, int hd_v, cudaStream_t stream) {
   if (n_ctx <= 0) return PTB_OK;
   if (heads <= 0 || dim <= 0 || rot_dim < 0 || vdim <= 0 || dim + rot_dim > hd || vdim > hd_v) return PTB_ERR_SIZE;
-  latent_unfold_kernel<<<n_ctx, 256, 0, stream>>>((const __nv_bfloat16*)kv, (const __nv_bfloat16*)kr_rows, *sb, ctx_seq,
-                                                  ctx_pos, (__nv_bfloat16*)k_tmp, (__nv_bfloat16*)v_tmp, heads, dim, rot_dim,
-                                                  vdim, hd, hd_v);
+  const bool words = dim % 8 == 0 && rot_dim % 8 == 0 && vdim % 8 == 0 && hd % 8 == 0 && hd_v % 8 == 0 && aligned16(kv) &&
+                     aligned16(kr_rows) && aligned16(k_tmp) && aligned16(v_tmp);
+#define PTB_UNFOLD(V)                                                                                                  \
+  latent_unfold_kernel<V><<<n_ctx, 256, 0, stream>>>((const __nv_bfloat16*)kv, (const __nv_bfloat16*)kr_rows, *sb, ctx_seq, \
+                                                     ctx_pos, (__nv_bfloat16*)k_tmp, (__nv_bfloat16*)v_tmp, heads, dim,    \
+                                                     rot_dim, vdim, hd, hd_v)
+  if (words) PTB_UNFOLD(8);
+  else PTB_UNFOLD(1);
+#undef PTB_UNFOLD
   return launch_status();
 }
 
@@ -806,17 +878,29 @@ PTB_API int ptb_latent_q_unfold(const void* q, long long q_stride, const float* 
   if (n_tokens <= 0) return PTB_OK;
   if (heads <= 0 || dim <= 0 || rot_dim < 0 || dim + rot_dim > hd || 2 * rot_pairs > rot_dim) return PTB_ERR_SIZE;
   if (rot_pairs > 0 && (rope_cos == nullptr || rope_sin == nullptr)) return PTB_ERR_SIZE;
-  latent_q_unfold_kernel<<<n_tokens, 256, 0, stream>>>((const __nv_bfloat16*)q, q_stride, rope_cos, rope_sin, rot_pairs, interleaved,
-                                                       (__nv_bfloat16*)out, heads, dim, rot_dim, hd);
+  const bool words = dim % 8 == 0 && rot_dim % 8 == 0 && hd % 8 == 0 && q_stride % 8 == 0 && aligned16(q) && aligned16(out);
+#define PTB_QUNFOLD(V)                                                                                                   \
+  latent_q_unfold_kernel<V><<<n_tokens, 256, 0, stream>>>((const __nv_bfloat16*)q, q_stride, rope_cos, rope_sin, rot_pairs, \
+                                                          interleaved, (__nv_bfloat16*)out, heads, dim, rot_dim, hd)
+  if (words) PTB_QUNFOLD(8);
+  else PTB_QUNFOLD(1);
+#undef PTB_QUNFOLD
   return launch_status();
 }
 
 PTB_API int ptb_gate_heads(const void* o, const void* gate, long long gate_t, void* out, int n_tokens, int heads, int vdim,
                            int hd, int per_head, cudaStream_t stream) {
-  const long long total = (long long)n_tokens * heads * vdim;
-  if (total <= 0) return PTB_OK;
-  const size_t want = (size_t(total) + 255) / 256, most = size_t(sm_count()) * 16;
-  gate_heads_kernel<<<int(want < most ? want : most), 256, 0, stream>>>((const __nv_bfloat16*)o, (const __nv_bfloat16*)gate,
-                                                                       gate_t, (__nv_bfloat16*)out, total, heads, vdim, hd, per_head);
+  if (n_tokens <= 0) return PTB_OK;
+  if (heads <= 0 || vdim <= 0 || hd < vdim) return PTB_ERR_SIZE;
+  const bool words = vdim % 8 == 0 && hd % 8 == 0 && aligned16(o) && aligned16(out);
+  const long long n = (long long)n_tokens * heads * (words ? vdim / 8 : vdim);
+  const size_t want = (size_t(n) + 255) / 256, most = size_t(sm_count()) * 16;
+  const int blocks = int(want < most ? want : most);
+#define PTB_GATE(V)                                                                                                     \
+  gate_heads_kernel<V><<<blocks, 256, 0, stream>>>((const __nv_bfloat16*)o, (const __nv_bfloat16*)gate, gate_t,          \
+                                                   (__nv_bfloat16*)out, n, heads, vdim, hd, per_head)
+  if (words) PTB_GATE(8);
+  else PTB_GATE(1);
+#undef PTB_GATE
   return launch_status();
 }

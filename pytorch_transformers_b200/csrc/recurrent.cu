@@ -6,7 +6,7 @@
 //   [0, R)                      the recurrence's state S
 //   [R + k R, R + (k + 1) R)    the convolution's input at position length - (taps - 1) + k, k < taps - 1
 // (zero for a sequence that has just started, which is the convolution's zero padding and S = 0).
-#include "common.cuh"
+#include "mma_common.cuh"
 
 namespace {
 
@@ -238,8 +238,9 @@ block_linear_kernel(const T* __restrict__ x, long long xt, long long xg, const T
   }
 }
 
-// The same for a few rows (steps of single tokens): a warp per (group, output) reads its row of W once,
-// lanes along K, and forms the sums of all M <= 16 rows; the order of a row's sums is fixed.
+// The same for a few rows (steps of single tokens): LANES lanes of a warp take SKINNY_R neighbouring outputs of a group,
+// each lane 8 consecutive k at a time, and form the sums of all M <= MT rows; a row of W is read once and a row of x once
+// for the SKINNY_R outputs. The order of a row's sums is fixed by K alone.
 constexpr int SKINNY_M = 16;
 template <typename T> __device__ __forceinline__ void load8(const T* p, float (&f)[8], bool vec);
 template <> __device__ __forceinline__ void load8<float>(const float* p, float (&f)[8], bool) {
@@ -256,53 +257,132 @@ template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bflo
 }
 
 // `vec`: every row of x and w starts on a 16-byte boundary and K is a multiple of 8 (the host checks):
-// bfloat16 operands then move in 16-byte words. A lane takes 8 consecutive k at a time.
-template <typename T, typename TO>
-__global__ void __launch_bounds__(256)
+// bfloat16 operands then move in 16-byte words.
+constexpr int SKINNY_R = 2, SKINNY_THREADS = 128;
+template <typename T, typename TO, int LANES, int MT>
+__global__ void __launch_bounds__(SKINNY_THREADS)
 block_linear_skinny_kernel(const T* __restrict__ x, long long xt, long long xg, const T* __restrict__ w,
                            const float* __restrict__ bias, TO* __restrict__ y, const T* __restrict__ gate,
                            long long gate_t, int gate_g, int gate_n, int M, int G, int N, int K, int act, int vec) {
-  const int lane = threadIdx.x % 32;
-  const long long item = (long long)blockIdx.x * (blockDim.x / 32) + threadIdx.x / 32;
-  if (item >= (long long)G * N) return;
-  const int g = int(item / N), n = int(item % N);
-  const T* wr = w + (size_t(g) * N + n) * K;
-  float acc[SKINNY_M];
+  const int lane = threadIdx.x % LANES;
+  const int per_group = (N + SKINNY_R - 1) / SKINNY_R;
+  const long long item = ((long long)blockIdx.x * SKINNY_THREADS + threadIdx.x) / LANES;
+  const bool mine = item < (long long)G * per_group;      // lanes past the end stay for the shuffles
+  const int g = mine ? int(item / per_group) : 0, n0 = mine ? int(item % per_group) * SKINNY_R : 0;
+  const T* wr[SKINNY_R];
 #pragma unroll
-  for (int m = 0; m < SKINNY_M; ++m) acc[m] = 0.f;
+  for (int r = 0; r < SKINNY_R; ++r) wr[r] = w + (size_t(g) * N + min(n0 + r, N - 1)) * K;
+  const T* xr = x + size_t(g) * xg;
+  float acc[SKINNY_R][MT];
+#pragma unroll
+  for (int r = 0; r < SKINNY_R; ++r)
+#pragma unroll
+    for (int m = 0; m < MT; ++m) acc[r][m] = 0.f;
   const int k_whole = K / 8 * 8;
-  for (int k = lane * 8; k < k_whole; k += 256) {
-    float wv[8];
-    load8<T>(wr + k, wv, vec);
+#pragma unroll 2
+  for (int k = lane * 8; k < k_whole; k += LANES * 8) {
+    float wv[SKINNY_R][8];
 #pragma unroll
-    for (int m = 0; m < SKINNY_M; ++m) {
+    for (int r = 0; r < SKINNY_R; ++r) load8<T>(wr[r] + k, wv[r], vec);
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
       if (m < M) {
         float xv[8];
-        load8<T>(x + size_t(m) * xt + size_t(g) * xg + k, xv, vec);
-        float part = 0.f;
+        load8<T>(xr + size_t(m) * xt + k, xv, vec);
 #pragma unroll
-        for (int i = 0; i < 8; ++i) part = fmaf(wv[i], xv[i], part);
-        acc[m] += part;
+        for (int r = 0; r < SKINNY_R; ++r) {
+          float part = 0.f;
+#pragma unroll
+          for (int i = 0; i < 8; ++i) part = fmaf(wv[r][i], xv[i], part);
+          acc[r][m] += part;
+        }
       }
     }
   }
-  for (int k = k_whole + lane; k < K; k += 32) {
-    const float wv = to_f(wr[k]);
+  for (int k = k_whole + lane; k < K; k += LANES) {
 #pragma unroll
-    for (int m = 0; m < SKINNY_M; ++m)
-      if (m < M) acc[m] = fmaf(wv, to_f(x[size_t(m) * xt + size_t(g) * xg + k]), acc[m]);
+    for (int m = 0; m < MT; ++m)
+      if (m < M) {
+        const float xv = to_f(xr[size_t(m) * xt + k]);
+#pragma unroll
+        for (int r = 0; r < SKINNY_R; ++r) acc[r][m] = fmaf(to_f(wr[r][k]), xv, acc[r][m]);
+      }
   }
 #pragma unroll
-  for (int m = 0; m < SKINNY_M; ++m) {
-    if (m >= M) break;
-    float v = warp_sum(acc[m]);
-    if (lane == 0) {
-      if (bias) v += bias[size_t(g) * N + n];
-      if (act == 1) v = 1.f / (1.f + expf(-v));
-      if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(m) * gate_t + size_t(g) * gate_g + size_t(n) * gate_n])));
-      y[(size_t(m) * G + g) * N + n] = from_f<TO>(v);
+  for (int r = 0; r < SKINNY_R; ++r) {
+#pragma unroll
+    for (int m = 0; m < MT; ++m) {
+      float v = acc[r][m];
+#pragma unroll
+      for (int o = LANES / 2; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+      const int n = n0 + r;
+      if (lane == m % LANES && m < M && mine && n < N) {      // every lane holds the sum: the rows' epilogues are shared out
+        if (bias) v += bias[size_t(g) * N + n];
+        if (act == 1) v = 1.f / (1.f + expf(-v));
+        if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(m) * gate_t + size_t(g) * gate_g + size_t(n) * gate_n])));
+        y[(size_t(m) * G + g) * N + n] = from_f<TO>(v);
+      }
     }
   }
+}
+
+// The same in bfloat16 on the tensor cores (mma.m16n8k16, float32 sums) for fewer rows than the library's batched product is
+// worth: a warp forms 16 rows x 8 outputs of a group over all of K, operands straight from global memory in 16-byte words. A
+// lane's word holds 8 consecutive k of its row; both operands take the same words in the same places, so the order of k inside
+// a group of 32 is permuted alike and every product meets its partner. Needs rows at whole 16-byte words, K a multiple of 8.
+template <typename TO>
+__global__ void __launch_bounds__(128)
+block_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, long long xt, long long xg, const __nv_bfloat16* __restrict__ w,
+                        const float* __restrict__ bias, TO* __restrict__ y, const __nv_bfloat16* __restrict__ gate,
+                        long long gate_t, int gate_g, int gate_n, int M, int G, int N, int K, int act) {
+  const int lane = threadIdx.x % 32, quad = lane % 4;
+  const int tiles = (N + 7) / 8;
+  const long long item = (long long)blockIdx.x * 4 + threadIdx.x / 32;
+  if (item >= (long long)G * tiles) return;
+  const int g = int(item / tiles), n0 = int(item % tiles) * 8, m0 = blockIdx.y * 16;
+  const int r_lo = m0 + lane / 4, r_hi = r_lo + 8, n = n0 + lane / 4;
+  const __nv_bfloat16* xl = x + size_t(r_lo < M ? r_lo : 0) * xt + size_t(g) * xg + quad * 8;
+  const __nv_bfloat16* xh = x + size_t(r_hi < M ? r_hi : 0) * xt + size_t(g) * xg + quad * 8;
+  const __nv_bfloat16* wn = w + (size_t(g) * N + (n < N ? n : 0)) * K + quad * 8;
+  const bool lo_ok = r_lo < M, hi_ok = r_hi < M, n_ok = n < N;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+  for (int k0 = 0; k0 < K; k0 += 32) {
+    const bool k_ok = k0 + quad * 8 < K;
+    const uint4 a = (k_ok && lo_ok) ? *reinterpret_cast<const uint4*>(xl + k0) : zero;
+    const uint4 b = (k_ok && hi_ok) ? *reinterpret_cast<const uint4*>(xh + k0) : zero;
+    const uint4 c = (k_ok && n_ok) ? *reinterpret_cast<const uint4*>(wn + k0) : zero;
+    const uint32_t a0[4] = {a.x, b.x, a.y, b.y}, a1[4] = {a.z, b.z, a.w, b.w};
+    mma_bf16(acc, a0, c.x, c.y);
+    mma_bf16(acc, a1, c.z, c.w);
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int m = i < 2 ? r_lo : r_hi, col = n0 + quad * 2 + (i & 1);
+    if (m >= M || col >= N) continue;
+    float v = acc[i];
+    if (bias) v += bias[size_t(g) * N + col];
+    if (act == 1) v = 1.f / (1.f + expf(-v));
+    if (gate) v *= 1.f / (1.f + expf(-to_f(gate[size_t(m) * gate_t + size_t(g) * gate_g + size_t(col) * gate_n])));
+    y[(size_t(m) * G + g) * N + col] = from_f<TO>(v);
+  }
+}
+
+template <typename T, typename TO, int MT>
+int launch_block_skinny(const void* x, long long xt, long long xg, const void* w, const float* bias, void* y, const void* gate,
+                        long long gate_t, int gate_g, int gate_n, int M, int G, int N, int K, int act, int vec,
+                        cudaStream_t stream) {
+  const long long items = (long long)G * ((N + SKINNY_R - 1) / SKINNY_R);
+#define PTB_BLS(LANES)                                                                                                     \
+  block_linear_skinny_kernel<T, TO, LANES, MT><<<int((items * LANES + SKINNY_THREADS - 1) / SKINNY_THREADS), SKINNY_THREADS, \
+                                                 0, stream>>>((const T*)x, xt, xg, (const T*)w, bias, (TO*)y, (const T*)gate, \
+                                                              gate_t, gate_g, gate_n, M, G, N, K, act, vec)
+  if (K <= 128) PTB_BLS(4);
+  else if (K <= 256) PTB_BLS(8);
+  else PTB_BLS(16);
+#undef PTB_BLS
+  return launch_status();
 }
 
 // The epilogue of block_linear for products that the library's batched routine made: z [groups, M, N]
@@ -415,20 +495,29 @@ PTB_API int ptb_block_linear(int dtype, int out_dtype, const void* x, long long 
   if (K <= 0 || act < 0 || act > 1 || G > 65535) return PTB_ERR_SIZE;
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM, G);
   if (grid.y > 65535) return PTB_ERR_SIZE;
-  if (M <= SKINNY_M) {
-    const long long items = (long long)G * N;
-    const int sgrid = int((items + 7) / 8);
-    typedef __nv_bfloat16 bf;
-    const int vec = (K % 8 == 0 && xt % 8 == 0 && xg % 8 == 0 && aligned16(x) && aligned16(w)) ? 1 : 0;
-    if (dtype == PTB_F32 && out_dtype == PTB_F32)
-      block_linear_skinny_kernel<float, float><<<sgrid, 256, 0, stream>>>((const float*)x, xt, xg, (const float*)w, bias, (float*)y, (const float*)gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec);
-    else if (dtype == PTB_BF16 && out_dtype == PTB_F32)
-      block_linear_skinny_kernel<bf, float><<<sgrid, 256, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (float*)y, (const bf*)gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec);
-    else if (dtype == PTB_BF16 && out_dtype == PTB_BF16)
-      block_linear_skinny_kernel<bf, bf><<<sgrid, 256, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (bf*)y, (const bf*)gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec);
+  typedef __nv_bfloat16 bf;
+  const int vec = (K % 8 == 0 && xt % 8 == 0 && xg % 8 == 0 && aligned16(x) && aligned16(w)) ? 1 : 0;
+  if (dtype == PTB_BF16 && vec) {
+    const dim3 mgrid(unsigned(((long long)G * ((N + 7) / 8) + 3) / 4), (M + 15) / 16);
+    if (mgrid.y > 65535) return PTB_ERR_SIZE;
+    if (out_dtype == PTB_F32)
+      block_linear_mma_kernel<float><<<mgrid, 128, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (float*)y, (const bf*)gate, gate_t, gate_g, gate_n, M, G, N, K, act);
+    else if (out_dtype == PTB_BF16)
+      block_linear_mma_kernel<bf><<<mgrid, 128, 0, stream>>>((const bf*)x, xt, xg, (const bf*)w, bias, (bf*)y, (const bf*)gate, gate_t, gate_g, gate_n, M, G, N, K, act);
     else
       return PTB_ERR_DTYPE;
     return launch_status();
+  }
+  if (M <= SKINNY_M) {
+#define PTB_BLM(TT, TTO)                                                                                                \
+  return M <= 4   ? launch_block_skinny<TT, TTO, 4>(x, xt, xg, w, bias, y, gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec, stream) \
+         : M <= 8 ? launch_block_skinny<TT, TTO, 8>(x, xt, xg, w, bias, y, gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec, stream) \
+                  : launch_block_skinny<TT, TTO, SKINNY_M>(x, xt, xg, w, bias, y, gate, gate_t, gate_g, gate_n, M, G, N, K, act, vec, stream)
+    if (dtype == PTB_F32 && out_dtype == PTB_F32) PTB_BLM(float, float);
+    if (dtype == PTB_BF16 && out_dtype == PTB_F32) PTB_BLM(bf, float);
+    if (dtype == PTB_BF16 && out_dtype == PTB_BF16) PTB_BLM(bf, bf);
+#undef PTB_BLM
+    return PTB_ERR_DTYPE;
   }
   if (dtype == PTB_F32 && out_dtype == PTB_F32)
     block_linear_kernel<float, float><<<grid, 256, 0, stream>>>((const float*)x, xt, xg, (const float*)w, bias,
