@@ -516,20 +516,33 @@ latent_attention_mma_kernel(const float* __restrict__ q_abs, const __nv_bfloat16
     }
     cp_async_wait<0>();
     __syncthreads();     // the page has landed for everybody (and the query rows are written)
-    // scores of keys 16 warp .. 16 warp + 15
+    // scores of keys 16 warp .. 16 warp + 15; four sums take turns (one alone would wait for each product in turn)
+    constexpr int CHAINS = 4;
+    float part_s[CHAINS][2][4];
+#pragma unroll
+    for (int u = 0; u < CHAINS; ++u)
+#pragma unroll
+      for (int f = 0; f < 2; ++f)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) part_s[u][f][c] = 0.f;
+    for (int ks0 = 0; ks0 < dk / 16; ks0 += CHAINS) {
+#pragma unroll
+      for (int u = 0; u < CHAINS; ++u) {
+        const int ks = ks0 + u;
+        if (ks >= dk / 16) continue;
+        uint32_t a[4], b0, b1, b2, b3;
+        ldmatrix_x4(a[0], a[1], a[2], a[3], q_base + (lane & 15) * rowb + (ks * 2 + (lane >> 4)) * 16);
+        const int id = lane >> 3;
+        ldmatrix_x4(b0, b1, b2, b3, k_base + (warp * 16 + (id >> 1) * 8 + (lane & 7)) * rowb + (ks * 2 + (id & 1)) * 16);
+        mma_bf16(part_s[u][0], a, b0, b1);
+        mma_bf16(part_s[u][1], a, b2, b3);
+      }
+    }
     float s[2][4];
 #pragma unroll
     for (int f = 0; f < 2; ++f)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) s[f][c] = 0.f;
-    for (int ks = 0; ks < dk / 16; ++ks) {
-      uint32_t a[4], b0, b1, b2, b3;
-      ldmatrix_x4(a[0], a[1], a[2], a[3], q_base + (lane & 15) * rowb + (ks * 2 + (lane >> 4)) * 16);
-      const int id = lane >> 3;
-      ldmatrix_x4(b0, b1, b2, b3, k_base + (warp * 16 + (id >> 1) * 8 + (lane & 7)) * rowb + (ks * 2 + (id & 1)) * 16);
-      mma_bf16(s[0], a, b0, b1);
-      mma_bf16(s[1], a, b2, b3);
-    }
+      for (int c = 0; c < 4; ++c) s[f][c] = (part_s[0][f][c] + part_s[1][f][c]) + (part_s[2][f][c] + part_s[3][f][c]);
     float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
     for (int f = 0; f < 2; ++f)
