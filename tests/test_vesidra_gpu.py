@@ -263,7 +263,7 @@ def test_latent_kernel_weights_in_two_terms(rank, rot, heads, tokens, splits):
 # ------------------------------------------------------------------------------------------------ the mixer
 MIXERS = [vm.mla(3, 40, 24, 36, 48, 0.15, 20000.0, (4.0, 60, 8.0, 1.0)),        # folded kernel: general; key rows of 64
           vm.mla(2, 64, 32, 96, 80, 0.1, 500.0),                               # tensor cores, five groups of columns; 128
-          vm.mla(4, 112, 48, 128, 128, 0.08, 50000.0, (8.0, 256, 16.0, 1.0)),  # key rows of 160 in 192
+          vm.mla(4, 112, 48, 128, 128, 0.08, 70000.0, (8.0, 256, 16.0, 1.0)),  # key rows of 160 in 192
           vm.mla(18, 32, 32, 64, 64, 0.125),                                   # more heads than a tile of one token has rows
           vm.mla(5, 7, 2, 9, 11, 0.4, 10.0), vm.mla(3, 10, 6, 14, 22, 0.3, 1000.0, (3.0, 77, 5.0, 0.5)),
           vm.mla(2, 150, 60, 40, 16, 0.08), vm.mla(1, 24, 16, 140, 32, 0.2),      # beyond the prompt kernel's sizes

@@ -88,7 +88,7 @@ def test_parts_refuse_what_their_kernels_do_not_take():
     from pytorch_transformers_b200 import kernels
     build = BuildContext(torch.device("cpu"), torch.float32, kernels)
     experts = dict(hidden=8, inner=4, experts=3, top=1)
-    for bad in (dict(experts, expert="plain"), dict(experts, weight_on="input"), dict(experts, score="tanh"),
+    for bad in (dict(experts, expert="plain", weight_on="both"), dict(experts, weight_on="input"), dict(experts, score="tanh"),
                 dict(experts, expert="plain", weight_on="input", identity=1, experts=2),
                 dict(experts, expert="plain", weight_on="input", activation="swish")):
         with pytest.raises(ValueError):

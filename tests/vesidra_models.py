@@ -63,7 +63,7 @@ CONFIGS = {
     ]),
     # sizes of the tensor cores: key rows of 160 entries beside values of 128, many heads, a latent of 256
     "wide": _cfg(310, 136, 11.0, 1e-5, [
-        (mla(4, 112, 48, 128, 128, 0.08, 50000.0, (8.0, 256, 16.0, 1.0)), moe(12, 3, 64, shared=96)),
+        (mla(4, 112, 48, 128, 128, 0.08, 70000.0, (8.0, 256, 16.0, 1.0)), moe(12, 3, 64, shared=96)),
         (mla(18, 32, 32, 64, 64, 0.125, 10000.0), dense(200)),
         (mla(6, 64, 64, 64, 256, 0.09, 1e5, (40.0, 512, 32.0, 1.0)), moe(4, 1, 48)),
     ]),
