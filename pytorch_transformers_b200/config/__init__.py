@@ -6,4 +6,5 @@ from .zalunex import ZalunexConfig
 from .pogezen import PogezenConfig
 from .figudra import FigudraConfig
 from .vesidra import VesidraConfig
+from .vabedra import VabedraConfig
 from .registry import AutoConfig, Architecture, lookup, lookup_config, register_architecture, registered

@@ -35,6 +35,16 @@ __device__ __forceinline__ float apply_activation(float v, int act) {
   }
 }
 
+// The unit between a gated feed-forward's two products: silu(gate) * up, or with limit > 0 the clamped unit
+// g * sigmoid(alpha g) * (u + 1) of g = min(gate, limit) and u = clamp(up, -limit, limit).
+__device__ __forceinline__ float gated_unit(float gate, float up, float limit, float alpha) {
+  if (limit > 0.f) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    return g / (1.f + expf(-alpha * g)) * (u + 1.f);
+  }
+  return gate / (1.f + expf(-gate)) * up;
+}
+
 // multiprocessors of the current device (asked once per process and device)
 inline int sm_count() {
   static int sms[64] = {};

@@ -270,7 +270,8 @@ expert_plan_kernel(const int* __restrict__ ids, int* __restrict__ plan, int pair
 }
 
 // Grouped product over the plan's tiles. MODE 0: rows are gathered from h by token (pair / top),
-// W [experts, 2 F, K] holds gate rows then up rows, out[row, f] = silu(gate) * up in the model dtype.
+// W [experts, 2 F, K] holds gate rows then up rows, out[row, f] = silu(gate) * up in the model dtype; with glu_limit > 0
+// the clamped unit instead: g = min(gate, limit), u = clamp(up, -limit, limit), out = g * sigmoid(glu_alpha g) * (u + 1).
 // MODE 1: rows are `x`'s sorted rows [pairs, K], W [experts, N, K], out [pairs, N] float32.
 // MODE 2: rows gathered from h as in MODE 0, W [experts, N, K] (an expert without a gate),
 // out[row, n] = act(row_scale[pair] * (W h)) in the model dtype: the expert's first product of the pair's
@@ -283,7 +284,7 @@ template <typename T, typename TO, int MODE, int TM>
 __global__ void __launch_bounds__(256)
 expert_linear_kernel(const T* __restrict__ x, const T* __restrict__ w, TO* __restrict__ out,
                      const int* __restrict__ plan, int pairs, int max_tiles, int top, int N, int K,
-                     const float* __restrict__ row_scale, int act) {
+                     const float* __restrict__ row_scale, int act, float glu_limit, float glu_alpha) {
   constexpr int EBM = TM * 16;
   const int tile = blockIdx.y;
   if (tile >= plan[0]) return;
@@ -353,7 +354,7 @@ expert_linear_kernel(const T* __restrict__ x, const T* __restrict__ w, TO* __res
       const int gn = n0 + tn + j;
       if (gn >= N) continue;
       float v = acc[0][i][j];
-      if (MODE == 0) v = v / (1.f + expf(-v)) * acc[MODE == 0 ? 1 : 0][i][j];
+      if (MODE == 0) v = gated_unit(v, acc[MODE == 0 ? 1 : 0][i][j], glu_limit, glu_alpha);
       if (MODE == 2) v = apply_activation(v * (row_scale ? row_scale[pair_of_row[row0 + tm + i]] : 1.f), act);
       out[size_t(row0 + tm + i) * N + gn] = from_f<TO>(v);
     }
@@ -388,14 +389,14 @@ __global__ void expert_combine_kernel(const TB* __restrict__ base, const T* __re
 
 template <typename T, typename TO, int MODE>
 int launch_expert_linear(const void* x, const void* w, void* out, const int* plan, int pairs, int max_tiles, int top,
-                         int N, int K, int tile_rows, const float* row_scale, int act, cudaStream_t stream) {
+                         int N, int K, int tile_rows, const float* row_scale, int act, float glu_limit, float glu_alpha, cudaStream_t stream) {
   dim3 grid((N + EBN - 1) / EBN, max_tiles);
   if (tile_rows == 16)
     expert_linear_kernel<T, TO, MODE, 1><<<grid, 256, 0, stream>>>((const T*)x, (const T*)w, (TO*)out, plan, pairs,
-                                                                   max_tiles, top, N, K, row_scale, act);
+                                                                   max_tiles, top, N, K, row_scale, act, glu_limit, glu_alpha);
   else if (tile_rows == 64)
     expert_linear_kernel<T, TO, MODE, 4><<<grid, 256, 0, stream>>>((const T*)x, (const T*)w, (TO*)out, plan, pairs,
-                                                                   max_tiles, top, N, K, row_scale, act);
+                                                                   max_tiles, top, N, K, row_scale, act, glu_limit, glu_alpha);
   else
     return PTB_ERR_SIZE;
   return launch_status();
@@ -469,16 +470,16 @@ PTB_API int ptb_expert_plan(const int* ids, int* plan, int pairs, int n_experts,
   return launch_status();
 }
 
-// mode 0: gate and up with silu(gate) * up, out in the model dtype; mode 1: down, out float32; mode 2: one product
+// mode 0: gate and up with silu(gate) * up (glu_limit > 0: the clamped unit), out in the model dtype; mode 1: down, out float32; mode 2: one product
 // with act(row_scale * .), out in the model dtype (row_scale [pairs] float32 or null, act: an activation code)
 PTB_API int ptb_expert_linear(int dtype, int mode, const void* x, const void* w, void* out, const int* plan, int pairs,
                               int max_tiles, int top, int N, int K, int tile_rows, const float* row_scale, int act,
-                              cudaStream_t stream) {
+                              float glu_limit, float glu_alpha, cudaStream_t stream) {
   if (pairs <= 0 || max_tiles <= 0) return PTB_OK;
   if (N <= 0 || K <= 0 || max_tiles > 65535 || top <= 0 || mode < 0 || mode > 2 || !activation_known(act))
     return PTB_ERR_SIZE;
 #define PTB_EL(TT, TTO, MM) \
-  launch_expert_linear<TT, TTO, MM>(x, w, out, plan, pairs, max_tiles, top, N, K, tile_rows, row_scale, act, stream)
+  launch_expert_linear<TT, TTO, MM>(x, w, out, plan, pairs, max_tiles, top, N, K, tile_rows, row_scale, act, glu_limit, glu_alpha, stream)
   if (dtype == PTB_F32) return mode == 0 ? PTB_EL(float, float, 0) : mode == 1 ? PTB_EL(float, float, 1) : PTB_EL(float, float, 2);
   if (dtype == PTB_BF16)
     return mode == 0 ? PTB_EL(__nv_bfloat16, __nv_bfloat16, 0)

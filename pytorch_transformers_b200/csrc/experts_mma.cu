@@ -4,7 +4,7 @@
 // tile and 64 of the 128 matrix rows. Operands come through a three-stage cp.async ring of [rows][32] tiles whose
 // 16-byte chunks are XOR-swizzled so that ldmatrix meets no bank twice.
 //   mode 0: x rows are gathered from h by token; the 128 matrix rows are 64 gate rows and the 64 up rows
-//           of the same columns; out[row, f] = silu(gate) * up, bfloat16.
+//           of the same columns; out[row, f] = silu(gate) * up (glu_limit > 0: the clamped unit, gated_unit), bfloat16.
 //   mode 1: x rows are the sorted rows themselves; out[row, n] float32.
 //   mode 2: x rows gathered as in mode 0, 128 plain matrix rows; out[row, n] = act(row_scale[pair] * sum), bfloat16
 //           (an expert without a gate; with row_scale its input is the token's row times the pair's weight).
@@ -24,7 +24,7 @@ template <int MODE, int GM>
 __global__ void __launch_bounds__(2 * GM)
 expert_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w, void* __restrict__ out_v,
                          const int* __restrict__ plan, int pairs, int max_tiles, int top, int N, int K,
-                         const float* __restrict__ row_scale, int act) {
+                         const float* __restrict__ row_scale, int act, float glu_limit, float glu_alpha) {
   const int tile = blockIdx.y;
   if (tile >= plan[0]) return;
   const int expert = plan[1 + tile], row0 = plan[1 + max_tiles + tile], rows = plan[1 + 2 * max_tiles + tile];
@@ -144,7 +144,7 @@ expert_linear_mma_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat1
             const int col = n0 + wn * 32 + j * 8 + c0 + q;
             if (col >= N) continue;
             const float g = acc[mi][j][half * 2 + q], u = acc[mi][j + 4][half * 2 + q];
-            o[col] = __float2bfloat16_rn(g / (1.f + expf(-g)) * u);
+            o[col] = __float2bfloat16_rn(gated_unit(g, u, glu_limit, glu_alpha));
           }
         }
       } else if (MODE == 2) {
@@ -181,7 +181,7 @@ PTB_API int ptb_expert_linear_mma_tile_rows() { return 64; }
 namespace {
 template <int MODE, int GM>
 int launch_expert_mma(const void* x, const void* w, void* out, const int* plan, int pairs, int max_tiles, int top, int N,
-                      int K, const float* row_scale, int act, cudaStream_t stream) {
+                      int K, const float* row_scale, int act, float glu_limit, float glu_alpha, cudaStream_t stream) {
   const size_t smem = size_t(STAGES) * (GM + GB) * 64 + GM * sizeof(int);
   static bool configured = false;
   if (!configured) {
@@ -192,7 +192,8 @@ int launch_expert_mma(const void* x, const void* w, void* out, const int* plan, 
   }
   dim3 grid((N + (MODE == 0 ? 63 : 127)) / (MODE == 0 ? 64 : 128), max_tiles);
   expert_linear_mma_kernel<MODE, GM><<<grid, 2 * GM, smem, stream>>>((const __nv_bfloat16*)x, (const __nv_bfloat16*)w, out,
-                                                                      plan, pairs, max_tiles, top, N, K, row_scale, act);
+                                                                      plan, pairs, max_tiles, top, N, K, row_scale, act, glu_limit,
+                                                                      glu_alpha);
   return launch_status();
 }
 }  // namespace
@@ -200,13 +201,13 @@ int launch_expert_mma(const void* x, const void* w, void* out, const int* plan, 
 // `tile_rows`: 64 or 128, the rows of the plan's tiles
 PTB_API int ptb_expert_linear_mma(int mode, const void* x, const void* w, void* out, const int* plan, int pairs,
                                   int max_tiles, int top, int N, int K, int tile_rows, const float* row_scale, int act,
-                                  cudaStream_t stream) {
+                                  float glu_limit, float glu_alpha, cudaStream_t stream) {
   if (pairs <= 0 || max_tiles <= 0) return PTB_OK;
   if (N <= 0 || K <= 0 || K % 8 != 0 || max_tiles > 65535 || top <= 0 || (tile_rows != 64 && tile_rows != 128) ||
       mode < 0 || mode > 2 || !activation_known(act))
     return PTB_ERR_SIZE;
   if (!aligned16(x) || !aligned16(w)) return PTB_ERR_ALIGN;
-#define PTB_EM(MM, GG) launch_expert_mma<MM, GG>(x, w, out, plan, pairs, max_tiles, top, N, K, row_scale, act, stream)
+#define PTB_EM(MM, GG) launch_expert_mma<MM, GG>(x, w, out, plan, pairs, max_tiles, top, N, K, row_scale, act, glu_limit, glu_alpha, stream)
   if (mode == 0) return tile_rows == 64 ? PTB_EM(0, 64) : PTB_EM(0, 128);
   if (mode == 2) return tile_rows == 64 ? PTB_EM(2, 64) : PTB_EM(2, 128);
   return tile_rows == 64 ? PTB_EM(1, 64) : PTB_EM(1, 128);

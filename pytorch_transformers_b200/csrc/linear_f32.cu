@@ -13,7 +13,7 @@ constexpr int TM = 4, TN = 4;             // outputs per thread; 256 threads
 
 __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict__ x, const float* __restrict__ w,
                                                          const float* __restrict__ bias, float* __restrict__ y, int M,
-                                                         int N, int K, int act) {
+                                                         int N, int K, int ldx, int act) {
   // k-major tiles: xs[k][m], ws[k][n]; +4 padding keeps the transposing stores off one bank
   __shared__ float xs[BK][BM + 4];
   __shared__ float ws[BK][BN + 4];
@@ -33,7 +33,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
     for (int q = 0; q < 4; ++q) {
       const int k = k0 + lk + q;
       const int gm = m0 + lrow, gn = n0 + lrow;
-      xs[lk + q][lrow] = (gm < M && k < K) ? x[size_t(gm) * K + k] : 0.f;
+      xs[lk + q][lrow] = (gm < M && k < K) ? x[size_t(gm) * ldx + k] : 0.f;
       ws[lk + q][lrow] = (gn < N && k < K) ? w[size_t(gn) * K + k] : 0.f;
     }
     __syncthreads();
@@ -79,12 +79,13 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(const float* __restrict
 
 }  // namespace
 
-PTB_API int ptb_linear_f32(const float* x, const float* w, const float* bias, float* y, int M, int N, int K, int act,
+// x [M, K] with rows ldx apart
+PTB_API int ptb_linear_f32(const float* x, const float* w, const float* bias, float* y, int M, int N, int K, int ldx, int act,
                            cudaStream_t stream) {
   if (M <= 0 || N <= 0) return PTB_OK;
-  if (K <= 0 || !activation_known(act)) return PTB_ERR_SIZE;
+  if (K <= 0 || ldx < K || !activation_known(act)) return PTB_ERR_SIZE;
   dim3 grid((N + BN - 1) / BN, (M + BM - 1) / BM);
   if (grid.y > 65535) return PTB_ERR_SIZE;
-  linear_f32_kernel<<<grid, 256, 0, stream>>>(x, w, bias, y, M, N, K, act);
+  linear_f32_kernel<<<grid, 256, 0, stream>>>(x, w, bias, y, M, N, K, ldx, act);
   return launch_status();
 }

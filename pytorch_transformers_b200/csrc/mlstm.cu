@@ -126,8 +126,8 @@ mlstm_scan_kernel(const T* __restrict__ proj, int stride, const float* __restric
 }
 
 // out[t][h][e] = x[t][h][e] / rms(x[t][h][:]) * gain[h * v_dim + e] * sigmoid(gate[t][h * v_dim + e]); a warp per (token, head)
-template <typename T>
-__global__ void head_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ gain, const T* __restrict__ gate,
+template <typename T, typename TG>
+__global__ void head_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ gain, const TG* __restrict__ gate,
                                       int gate_stride, T* __restrict__ out, int out_stride, int n, int heads, int v_dim,
                                       float eps, int gate_silu) {
   const int warp = (blockIdx.x * blockDim.x + threadIdx.x) / 32, lane = threadIdx.x % 32;
@@ -199,21 +199,22 @@ PTB_API int ptb_mlstm_state_floats(int heads, int dim, int v_dim) {
   return heads * (dim * v_dim + ((v_dim + VB - 1) / VB) * (dim + 1));
 }
 
-// x float32 [n, heads * v_dim]; gain float32 [heads * v_dim]; gate (may be null) and out of `dtype`, rows gate_stride and
-// out_stride apart.
-PTB_API int ptb_head_norm_gate_act(const float* x, const float* gain, int dtype, const void* gate, int gate_stride, void* out,
-                               int out_stride, int n, int heads, int v_dim, float eps, int gate_silu, cudaStream_t stream) {
+// x float32 [n, heads * v_dim]; gain float32 [heads * v_dim]; gate (may be null; of gate_dtype: `dtype` or float32) and out of
+// `dtype`, rows gate_stride and out_stride apart.
+PTB_API int ptb_head_norm_gate_act(const float* x, const float* gain, int dtype, int gate_dtype, const void* gate, int gate_stride,
+                                   void* out, int out_stride, int n, int heads, int v_dim, float eps, int gate_silu, cudaStream_t stream) {
   if (n <= 0) return PTB_OK;
   if (heads <= 0 || v_dim <= 0 || out_stride < heads * v_dim) return PTB_ERR_SIZE;
   const long long warps = (long long)n * heads;
   const int threads = 256;
   const unsigned blocks = unsigned((warps * 32 + threads - 1) / threads);
-  if (dtype == PTB_F32)
-    head_norm_gate_kernel<float><<<blocks, threads, 0, stream>>>(x, gain, (const float*)gate, gate_stride, (float*)out,
-                                                                 out_stride, n, heads, v_dim, eps, gate_silu);
-  else if (dtype == PTB_BF16)
-    head_norm_gate_kernel<__nv_bfloat16><<<blocks, threads, 0, stream>>>(x, gain, (const __nv_bfloat16*)gate, gate_stride,
-                                                                         (__nv_bfloat16*)out, out_stride, n, heads, v_dim, eps, gate_silu);
+#define PTB_HNG(TT, TG)                                                                                                  \
+  head_norm_gate_kernel<TT, TG><<<blocks, threads, 0, stream>>>(x, gain, (const TG*)gate, gate_stride, (TT*)out, out_stride, \
+                                                                n, heads, v_dim, eps, gate_silu)
+  if (dtype == PTB_F32 && gate_dtype == PTB_F32) PTB_HNG(float, float);
+  else if (dtype == PTB_BF16 && gate_dtype == PTB_BF16) PTB_HNG(__nv_bfloat16, __nv_bfloat16);
+  else if (dtype == PTB_BF16 && gate_dtype == PTB_F32) PTB_HNG(__nv_bfloat16, float);
+#undef PTB_HNG
   else
     return PTB_ERR_DTYPE;
   return launch_status();
@@ -221,5 +222,5 @@ PTB_API int ptb_head_norm_gate_act(const float* x, const float* gain, int dtype,
 
 PTB_API int ptb_head_norm_gate(const float* x, const float* gain, int dtype, const void* gate, int gate_stride, void* out,
                                int out_stride, int n, int heads, int v_dim, float eps, cudaStream_t stream) {
-  return ptb_head_norm_gate_act(x, gain, dtype, gate, gate_stride, out, out_stride, n, heads, v_dim, eps, 0, stream);
+  return ptb_head_norm_gate_act(x, gain, dtype, dtype, gate, gate_stride, out, out_stride, n, heads, v_dim, eps, 0, stream);
 }

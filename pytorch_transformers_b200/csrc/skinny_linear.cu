@@ -78,7 +78,7 @@ template <int MT, int NT, int UNROLL>
 __global__ void __launch_bounds__(WARPS * 32)
 skinny_linear_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __restrict__ w,
                      const float* __restrict__ bias, const __nv_bfloat16* __restrict__ add,
-                     __nv_bfloat16* __restrict__ y_bf16, float* __restrict__ y_f32, int M, int N, int K, int act,
+                     __nv_bfloat16* __restrict__ y_bf16, float* __restrict__ y_f32, int M, int N, int K, int ldx, int act,
                      int ksplit, float* __restrict__ scratch, int* __restrict__ tickets) {
   __shared__ float red[WARPS][MT * 16][NT * 8 + 1];
   __shared__ int is_last;
@@ -105,7 +105,7 @@ skinny_linear_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* _
 #pragma unroll
   for (int j = 0; j < NT; ++j) {
     xok[j] = (j * 8 + g) < M;
-    xrow[j] = x + size_t(xok[j] ? j * 8 + g : 0) * K + t * 8;
+    xrow[j] = x + size_t(xok[j] ? j * 8 + g : 0) * ldx + t * 8;
   }
 
   // The warps take the 32-wide chunks of K in turn, UNROLL chunks at a time: at any moment the block
@@ -200,7 +200,7 @@ int k_split(int tiles, int chunks, int round) {
 
 template <int MT, int NT, int U>
 int launch_skinny(const void* x, const void* w, const float* bias, const void* add, void* y_bf16, float* y_f32,
-                  int M, int N, int K, int act, float* scratch, size_t scratch_floats, int* tickets, int n_tickets,
+                  int M, int N, int K, int ldx, int act, float* scratch, size_t scratch_floats, int* tickets, int n_tickets,
                   size_t* need_floats, cudaStream_t stream) {
   const int tiles = (N + 16 * MT - 1) / (16 * MT);
   int ksplit = k_split(tiles, K / KC, WARPS * U);
@@ -212,12 +212,12 @@ int launch_skinny(const void* x, const void* w, const float* bias, const void* a
   if (scratch == nullptr || tickets == nullptr || scratch_floats < need || n_tickets < tiles) ksplit = 1;
   skinny_linear_kernel<MT, NT, U><<<tiles * ksplit, WARPS * 32, 0, stream>>>(
       (const __nv_bfloat16*)x, (const __nv_bfloat16*)w, bias, (const __nv_bfloat16*)add, (__nv_bfloat16*)y_bf16,
-      y_f32, M, N, K, act, ksplit, scratch, tickets);
+      y_f32, M, N, K, ldx, act, ksplit, scratch, tickets);
   return launch_status();
 }
 
 int dispatch_skinny(const void* x, const void* w, const float* bias, const void* add, void* y_bf16, float* y_f32, int M,
-                    int N, int K, int act, float* scratch, size_t scratch_floats, int* tickets, int n_tickets,
+                    int N, int K, int ldx, int act, float* scratch, size_t scratch_floats, int* tickets, int n_tickets,
                     size_t* need_floats, cudaStream_t stream) {
   // Tile height and chunks in flight per warp, from a sweep over matrices of 4,096 to 65,024 rows (each
   // alone, from HBM): matrices with four tiles or more per SM (many rows, short K) want 32 rows per
@@ -225,7 +225,7 @@ int dispatch_skinny(const void* x, const void* w, const float* bias, const void*
   // the others 16 rows and four chunks.
   const bool wide = N >= 16 * sm_count() * 4;   // four 16-row tiles or more per SM
 #define PTB_SKINNY(MT, NT, U) \
-  return launch_skinny<MT, NT, U>(x, w, bias, add, y_bf16, y_f32, M, N, K, act, scratch, scratch_floats, tickets, \
+  return launch_skinny<MT, NT, U>(x, w, bias, add, y_bf16, y_f32, M, N, K, ldx, act, scratch, scratch_floats, tickets, \
                                   n_tickets, need_floats, stream)
   if (M <= 8) {
     if (wide) PTB_SKINNY(2, 1, 4);
@@ -246,26 +246,26 @@ int dispatch_skinny(const void* x, const void* w, const float* bias, const void*
 PTB_API int ptb_skinny_linear_max_rows() { return 32; }
 PTB_API int ptb_skinny_linear_k_multiple() { return KC; }
 
-// y = act(x w^T + bias) + add. x [M, K], w [N, K], add [M, N] bfloat16; bias float32 [N];
+// y = act(x w^T + bias) + add. x [M, K] (rows ldx apart, whole 16-byte words), w [N, K], add [M, N] bfloat16; bias float32 [N];
 // exactly one of y_bf16, y_f32 is given. M <= 32, K a multiple of 32, 16-byte aligned x and w.
 // scratch (float32, scratch_floats of them) and tickets (int32, n_tickets of them, all zero between
 // launches: the kernel puts them back) let the kernel divide K among several blocks per tile where that
 // balances the SMs; without them it does not divide. ptb_skinny_linear_scratch says how many floats a
 // launch would use.
 PTB_API int ptb_skinny_linear(const void* x, const void* w, const float* bias, const void* add, void* y_bf16,
-                              float* y_f32, int M, int N, int K, int act, float* scratch, size_t scratch_floats,
+                              float* y_f32, int M, int N, int K, int ldx, int act, float* scratch, size_t scratch_floats,
                               int* tickets, int n_tickets, cudaStream_t stream) {
   if (M <= 0 || N <= 0) return PTB_OK;
-  if (M > 32 || K <= 0 || K % KC != 0 || !activation_known(act)) return PTB_ERR_SIZE;
+  if (M > 32 || K <= 0 || K % KC != 0 || ldx < K || !activation_known(act)) return PTB_ERR_SIZE;
   if ((y_bf16 == nullptr) == (y_f32 == nullptr)) return PTB_ERR_SIZE;
-  if ((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) return PTB_ERR_ALIGN;
-  return dispatch_skinny(x, w, bias, add, y_bf16, y_f32, M, N, K, act, scratch, scratch_floats, tickets, n_tickets,
+  if (((reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(w)) & 15) || ldx % 8 != 0) return PTB_ERR_ALIGN;
+  return dispatch_skinny(x, w, bias, add, y_bf16, y_f32, M, N, K, ldx, act, scratch, scratch_floats, tickets, n_tickets,
                          nullptr, stream);
 }
 
 PTB_API long long ptb_skinny_linear_scratch(int M, int N, int K) {
   if (M <= 0 || N <= 0 || M > 32 || K <= 0 || K % KC != 0) return 0;
   size_t need = 0;
-  dispatch_skinny(nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, M, N, K, 0, nullptr, 0, nullptr, 0, &need, nullptr);
+  dispatch_skinny(nullptr, nullptr, nullptr, nullptr, nullptr, nullptr, M, N, K, K, 0, nullptr, 0, nullptr, 0, &need, nullptr);
   return (long long)need;
 }

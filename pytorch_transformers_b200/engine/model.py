@@ -82,6 +82,7 @@ class CausalLM:
         self.embedding: Optional[torch.Tensor] = None
         self.head: Optional[torch.Tensor] = None
         self.position_table: Optional[torch.Tensor] = None
+        self.token_table: Optional[torch.Tensor] = None
         if spec.position_table_name is not None and not (spec.stream_float32 and spec.max_positions > 0):
             raise ValueError("a learned position table needs a float32 stream and max_positions > 0")
         self.status = None  # device int32 word raised by kernels that clamp a bad index
@@ -114,6 +115,8 @@ class CausalLM:
             table[self.spec.head_name] = (None, "head", ParamDecl((v, h)))
         if self.spec.position_table_name is not None:
             table[self.spec.position_table_name] = (None, "positions", ParamDecl((self.spec.max_positions, h)))
+        if self.spec.token_table_name is not None:
+            table[self.spec.token_table_name] = (None, "token_table", ParamDecl((v, self.spec.token_table_width), std=1.0))
         for top in self._top_parts():
             for part in top.walk():
                 for logical, decl in part.param_decls().items():
@@ -144,6 +147,8 @@ class CausalLM:
                     self.embedding = t
                 elif logical == "positions":
                     self.position_table = t
+                elif logical == "token_table":
+                    self.token_table = t
                 else:
                     self.head = t
             else:
@@ -160,7 +165,7 @@ class CausalLM:
 
     def weight_bytes(self) -> int:
         seen, total = set(), 0
-        tensors = [self.embedding, self.head, self.position_table]
+        tensors = [self.embedding, self.head, self.position_table, self.token_table]
         for top in self._top_parts():
             for part in top.walk():
                 tensors += [getattr(part, a) for a in vars(part) if a.startswith("p_")]
@@ -373,6 +378,7 @@ class CausalLM:
     def forward(self, ctx: StepContext) -> torch.Tensor:
         k = self.build.kernels
         ctx.begin_forward()
+        ctx.token_table, ctx.status = self.token_table, self.status
         if self._two_streams(ctx):
             if self._side_stream is None:
                 self._side_stream = torch.cuda.Stream(device=self.device)

@@ -110,7 +110,8 @@ def lib():
                      "ptb_mlstm_chunk_tokens", "ptb_embed_rows", "ptb_attention_generic_capped", "ptb_attention_mma_capped",
                      "ptb_qk_prepare_store", "ptb_route_grouped", "ptb_expert_combine_shared", "ptb_glu_act",
                      "ptb_head_norm_gate_act", "ptb_gla_decay", "ptb_gla_walk", "ptb_gla_chunks", "ptb_gla_max_dim",
-                     "ptb_gla_chunk_tokens", "ptb_route_biased", "ptb_attention_tc_sizes", "ptb_attention_tc_supports_sizes"):
+                     "ptb_gla_chunk_tokens", "ptb_delta_prepare", "ptb_delta_walk", "ptb_delta_chunks",
+                     "ptb_delta_chunks_supports", "ptb_post_norm", "ptb_token_gate", "ptb_round_rows", "ptb_route_biased", "ptb_attention_tc_sizes", "ptb_attention_tc_supports_sizes"):
             getattr(L, name).restype = ctypes.c_int
         L.ptb_latent_part_floats.restype = ctypes.c_longlong
         L.ptb_expert_plan_words.restype = ctypes.c_longlong
@@ -209,8 +210,9 @@ def fill_normal(out: torch.Tensor, key: int, std: float, offset: float = 0.0, fi
 
 
 def linear_f32(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, act: str = "none"):
-    """act(x @ w.T + bias) in true float32 on the CUDA cores."""
-    _need_cuda(x, w, bias)
+    """act(x @ w.T + bias) in true float32 on the CUDA cores (the rows of x may lie wider apart)."""
+    _need_cuda(w, bias)
+    _check_rows(x, x.shape, torch.float32, "linear_f32: x")
     if x.dtype != torch.float32 or w.dtype != torch.float32:
         raise KernelError("linear_f32 takes float32 tensors")
     m, k = x.shape
@@ -218,7 +220,8 @@ def linear_f32(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = 
     if w.shape[1] != k:
         raise KernelError(f"linear_f32: x is [{m}, {k}] but w is {list(w.shape)}")
     y = torch.empty((m, n), dtype=torch.float32, device=x.device)
-    _check(lib().ptb_linear_f32(_ptr(x), _ptr(w), _ptr(bias), _ptr(y), m, n, k, ACTIVATIONS[act], _stream(x)),
+    _check(lib().ptb_linear_f32(_ptr(x), _ptr(w), _ptr(bias), _ptr(y), m, n, k, x.stride(0) if m > 1 else k, ACTIVATIONS[act],
+                               _stream(x)),
            "linear_f32")
     return y
 
@@ -677,8 +680,10 @@ def skinny_linear_preferred(rows: int, k: int, n: int = 0) -> bool:
 def skinny_linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, act: str = "none",
                   add: Optional[torch.Tensor] = None, out_dtype: torch.dtype = torch.bfloat16) -> torch.Tensor:
     """act(x @ w.T + bias) + add for up to 32 rows of bfloat16 x: one pass over w at memory speed,
-    float32 accumulation and epilogue; the result is bfloat16 or float32."""
-    _need_cuda(x, w, bias, add)
+    float32 accumulation and epilogue; the result is bfloat16 or float32. The rows of x may lie wider apart (a slice of
+    columns that starts and steps at whole 16-byte words)."""
+    _need_cuda(w, bias, add)
+    _check_rows(x, x.shape, torch.bfloat16, "skinny_linear: x")
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or (add is not None and add.dtype != torch.bfloat16):
         raise KernelError("skinny_linear takes bfloat16 x, w and add")
     m, k = x.shape
@@ -694,6 +699,7 @@ def skinny_linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor]
     n_tickets = (n + 15) // 16 if need else 0        # a ticket per tile of weight rows; tiles have 16 rows or more
     tickets = _tickets(n_tickets, x.device) if need else None
     _check(lib().ptb_skinny_linear(_ptr(x), _ptr(w), _ptr(bias), _ptr(add), _ptr(ybf), _ptr(yf), m, n, k,
+                                   x.stride(0) if m > 1 else k,
                                    ACTIVATIONS[act], _ptr(scratch), ctypes.c_size_t(need), _ptr(tickets),
                                    n_tickets, _stream(x)), "skinny_linear")
     return y
@@ -779,7 +785,8 @@ def matmul_nt(x: torch.Tensor, w: torch.Tensor, out_dtype: Optional[torch.dtype]
     its own kernel (linear_f32)."""
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16:
         raise KernelError("matmul_nt is the bfloat16 library product; float32 goes through linear_f32")
-    _need_cuda(x, w)
+    _need_cuda(w)
+    _check_rows(x, x.shape, torch.bfloat16, "matmul_nt: x")      # rows may lie wider apart
     if add is not None:
         # the library's own epilogue adds in float32 and rounds once (beta = 1)
         if out_dtype not in (None, torch.bfloat16) or add.dtype != torch.bfloat16 or tuple(add.shape) != (x.shape[0], w.shape[0]):
@@ -1072,33 +1079,21 @@ def route(h: torch.Tensor, w_router: torch.Tensor, correction: Optional[torch.Te
     return (ids, gates, logits) if extra else (ids, gates)
 
 
-def routed_experts(h: torch.Tensor, ids: torch.Tensor, gates: torch.Tensor, w_gate_up: torch.Tensor,
-                   w_down: torch.Tensor, base: Optional[torch.Tensor] = None, mma_tile_rows: int = 0,
-                   plain_act: Optional[str] = None, shared: Optional[torch.Tensor] = None,
-                   shared_gate: Optional[torch.Tensor] = None, weigh_output: bool = False) -> torch.Tensor:
-    """base + sum over a token's choices of weight * expert(h): experts ``w_gate_up`` [E, 2 F, width]
-    (gate rows, then up rows) and ``w_down`` [E, width, F] compute down(silu(gate h) * (up h)); an id >= E
-    is an identity expert. Pairs are sorted by expert on the device and run as tiles of grouped
-    products. Returns [tokens, width] in ``base``'s dtype (float32 without a base).
-
-    With ``plain_act`` (an activation's name) the experts have no gate and take their weight on the input:
-    ``w_gate_up`` is [E, F, width] and the result is base + sum of down(act(up (weight * h))); with ``weigh_output``
-    they too take it on the output, base + sum of weight * down(act(up h)).
-
-    ``shared`` (float32 [tokens, width]): the result of an expert that every token uses, added in the same kernel, times
-    sigmoid(``shared_gate``) where that is given (float32 [tokens, 1], a view whose rows may lie wider apart)."""
-    _need_cuda(h, ids, gates, w_gate_up, w_down, base, shared)
-    if shared is not None and (shared.dtype != torch.float32 or shared.shape != h.shape):
-        raise KernelError("routed_experts: the shared expert's rows are float32 [tokens, width]")
-    if shared_gate is not None and (shared is None or shared_gate.dtype != torch.float32 or shared_gate.shape[0] != h.shape[0]):
-        raise KernelError("routed_experts: the shared expert's gate is one float32 logit per token")
+def expert_rows(h: torch.Tensor, ids: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, mma_tile_rows: int = 0,
+                plain_act: Optional[str] = None, input_weights: Optional[torch.Tensor] = None, clamp=None):
+    """The chosen experts' results before they are summed: (float32 rows [tokens * top, width] sorted by expert, int32
+    [tokens * top]: the row of each (token, choice), -1 for an identity expert). Arguments as ``routed_experts`` takes them;
+    ``input_weights``: the weights [tokens, top] that plain experts take on their input."""
+    _need_cuda(h, ids, w_gate_up, w_down, input_weights)
     n_tokens, width = h.shape
     top = ids.shape[1]
     n_experts, two_f, _ = w_gate_up.shape
     f = two_f // 2 if plain_act is None else two_f
     first, act = (0, 0) if plain_act is None else (2, ACTIVATIONS[plain_act])
-    on_input = plain_act is not None and not weigh_output
-    scale = gates if on_input else None
+    scale = input_weights
+    if clamp is not None and (plain_act is not None or not clamp[0] > 0):
+        raise KernelError("expert_rows: a clamped unit belongs to gated experts and has a positive limit")
+    limit, alpha = (ctypes.c_float(clamp[0]), ctypes.c_float(clamp[1])) if clamp is not None else (ctypes.c_float(0), ctypes.c_float(0))
     pairs = n_tokens * top
     # bfloat16 with row sizes in whole 16-byte words: the tensor-core kernel (tiles of 64 rows); else float32 FMAs
     mma = h.dtype == torch.bfloat16 and width % 8 == 0 and f % 8 == 0
@@ -1120,22 +1115,52 @@ def routed_experts(h: torch.Tensor, ids: torch.Tensor, gates: torch.Tensor, w_ga
     y = torch.empty((pairs, width), dtype=torch.float32, device=h.device)
     if mma:
         _check(L.ptb_expert_linear_mma(first, _ptr(h), _ptr(w_gate_up), _ptr(a), _ptr(plan), pairs, max_tiles, top, f, width,
-                                       tile_rows, _ptr(scale), act, stream), "expert_linear_mma (gate, up)")
+                                       tile_rows, _ptr(scale), act, limit, alpha, stream), "expert_linear_mma (gate, up)")
         _check(L.ptb_expert_linear_mma(1, _ptr(a), _ptr(w_down), _ptr(y), _ptr(plan), pairs, max_tiles, top, width, f,
-                                       tile_rows, None, 0, stream), "expert_linear_mma (down)")
+                                       tile_rows, None, 0, ctypes.c_float(0), ctypes.c_float(0), stream), "expert_linear_mma (down)")
     else:
         _check(L.ptb_expert_linear(code, first, _ptr(h), _ptr(w_gate_up), _ptr(a), _ptr(plan), pairs, max_tiles, top, f, width,
-                                   tile_rows, _ptr(scale), act, stream), "expert_linear (gate, up)")
+                                   tile_rows, _ptr(scale), act, limit, alpha, stream), "expert_linear (gate, up)")
         _check(L.ptb_expert_linear(code, 1, _ptr(a), _ptr(w_down), _ptr(y), _ptr(plan), pairs, max_tiles, top, width, f,
-                                   tile_rows, None, 0, stream), "expert_linear (down)")
+                                   tile_rows, None, 0, ctypes.c_float(0), ctypes.c_float(0), stream), "expert_linear (down)")
+    return y, plan[1 + 3 * max_tiles:1 + 3 * max_tiles + pairs]
+
+
+def routed_experts(h: torch.Tensor, ids: torch.Tensor, gates: torch.Tensor, w_gate_up: torch.Tensor,
+                   w_down: torch.Tensor, base: Optional[torch.Tensor] = None, mma_tile_rows: int = 0,
+                   plain_act: Optional[str] = None, shared: Optional[torch.Tensor] = None,
+                   shared_gate: Optional[torch.Tensor] = None, weigh_output: bool = False,
+                   clamp=None) -> torch.Tensor:
+    """base + sum over a token's choices of weight * expert(h): experts ``w_gate_up`` [E, 2 F, width]
+    (gate rows, then up rows) and ``w_down`` [E, width, F] compute down(silu(gate h) * (up h)); an id >= E
+    is an identity expert. Pairs are sorted by expert on the device and run as tiles of grouped
+    products. Returns [tokens, width] in ``base``'s dtype (float32 without a base).
+
+    With ``plain_act`` (an activation's name) the experts have no gate and take their weight on the input:
+    ``w_gate_up`` is [E, F, width] and the result is base + sum of down(act(up (weight * h))); with ``weigh_output``
+    they too take it on the output, base + sum of weight * down(act(up h)).
+
+    ``clamp`` = (limit, alpha): the gated experts' unit is g * sigmoid(alpha g) * (u + 1) with g = min(gate h, limit) and
+    u = clamp(up h, -limit, limit).
+
+    ``shared`` (float32 [tokens, width]): the result of an expert that every token uses, added in the same kernel, times
+    sigmoid(``shared_gate``) where that is given (float32 [tokens, 1], a view whose rows may lie wider apart)."""
+    _need_cuda(h, ids, gates, w_gate_up, w_down, base, shared)
+    if shared is not None and (shared.dtype != torch.float32 or shared.shape != h.shape):
+        raise KernelError("routed_experts: the shared expert's rows are float32 [tokens, width]")
+    if shared_gate is not None and (shared is None or shared_gate.dtype != torch.float32 or shared_gate.shape[0] != h.shape[0]):
+        raise KernelError("routed_experts: the shared expert's gate is one float32 logit per token")
+    n_tokens, width = h.shape
+    top = ids.shape[1]
+    on_input = plain_act is not None and not weigh_output
+    y, row_of_pair = expert_rows(h, ids, w_gate_up, w_down, mma_tile_rows, plain_act, gates if on_input else None, clamp)
     if base is not None and (base.shape != h.shape or base.dtype not in (torch.float32, h.dtype)):
         raise KernelError("routed_experts: base must have the input's shape, in float32 or the input's dtype")
     out = torch.empty((n_tokens, width), dtype=torch.float32 if base is None else base.dtype, device=h.device)
-    row_of_pair = plan[1 + 3 * max_tiles:1 + 3 * max_tiles + pairs]
-    _check(L.ptb_expert_combine_shared(code, _dtype_code(out), _ptr(base), _ptr(h), _ptr(y), _ptr(ids),
+    _check(lib().ptb_expert_combine_shared(_dtype_code(h), _dtype_code(out), _ptr(base), _ptr(h), _ptr(y), _ptr(ids),
                                        _ptr(None if on_input else gates),
                                        _ptr(row_of_pair), _ptr(out), n_tokens, width, top, _ptr(shared), _ptr(shared_gate),
-                                       0 if shared_gate is None else shared_gate.stride(0), stream), "expert_combine")
+                                       0 if shared_gate is None else shared_gate.stride(0), _stream(h)), "expert_combine")
     return out
 
 
@@ -1403,20 +1428,24 @@ def mlstm(proj: torch.Tensor, gates: torch.Tensor, bias_i: torch.Tensor, bias_f:
 
 
 def head_norm_gate(x: torch.Tensor, gain: torch.Tensor, gate: Optional[torch.Tensor], heads: int, eps: float,
-                   out_dtype: torch.dtype, gate_act: str = "sigmoid") -> torch.Tensor:
+                   out_dtype: torch.dtype, gate_act: str = "sigmoid", out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Every head's stretch of the float32 rows ``x`` [tokens, heads * v_dim] divided by its root mean square, times
     ``gain`` [heads * v_dim] times sigmoid(``gate``) (of ``out_dtype``; rows may lie wider apart), in ``out_dtype``.
-    ``gate_act`` "silu": times gate * sigmoid(gate) instead."""
+    ``gate_act`` "silu": times gate * sigmoid(gate) instead. The gate may be float32 as well; ``out``: a
+    [tokens, heads * v_dim] view (rows may lie wider apart) to write into."""
     if gate_act not in ("sigmoid", "silu"):
         raise KernelError(f"head_norm_gate: the gate's activation is 'sigmoid' or 'silu', got {gate_act!r}")
     _need_cuda(x, gain)
     n, width = x.shape
     if x.dtype != torch.float32 or width % heads or gain.dtype != torch.float32 or gain.numel() != width:
         raise KernelError("head_norm_gate takes float32 rows [tokens, heads * v_dim] and a float32 gain of that width")
-    out = torch.empty((n, width), dtype=out_dtype, device=x.device)
+    if out is None:
+        out = torch.empty((n, width), dtype=out_dtype, device=x.device)
+    _check_rows(out, (n, width), out_dtype, "head_norm_gate: out")
     if gate is not None:
-        _check_rows(gate, (n, width), out_dtype, "head_norm_gate: gate")
-    _check(lib().ptb_head_norm_gate_act(_ptr(x), _ptr(gain), _dtype_code(out), _ptr(gate),
+        _check_rows(gate, (n, width), torch.float32 if gate.dtype == torch.float32 else out_dtype, "head_norm_gate: gate")
+    _check(lib().ptb_head_norm_gate_act(_ptr(x), _ptr(gain), _dtype_code(out),
+                                        _dtype_code(out if gate is None else gate), _ptr(gate),
                                         0 if gate is None else gate.stride(0), _ptr(out), out.stride(0), n, heads,
                                         width // heads, ctypes.c_float(eps), 1 if gate_act == "silu" else 0, _stream(x)),
            "head_norm_gate")
@@ -1469,4 +1498,164 @@ def gla(proj: torch.Tensor, log_decay: torch.Tensor, state: torch.Tensor, slots:
                                 _stream(proj)), "gla_chunks")
     global launches
     launches += 2       # three kernels
+    return out
+
+
+# ------------------------------------------------------------------------------------------------
+# The gated delta rule
+DELTA_MAX_DIM = 256   # ptb_delta_max_dim()
+DELTA_MAX_TAPS = 8    # ptb_delta_max_taps()
+DELTA_CHUNK = 64      # ptb_delta_chunk_tokens()
+
+
+def delta_state_floats(heads: int, kv_heads: int, dim: int, v_dim: int, taps: int) -> int:
+    """Per sequence: the convolution's last inputs, then S; whole 16-byte words."""
+    return ((taps - 1) * (2 * kv_heads * dim + heads * v_dim) + heads * dim * v_dim + 3) // 4 * 4
+
+
+def delta_prepare(proj: torch.Tensor, conv: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, batch: StepBatchC,
+                  a_log: torch.Tensor, dt_bias: torch.Tensor, heads: int, kv_heads: int, dim: int, v_dim: int, b_off: int,
+                  a_off: int = 0, z: Optional[torch.Tensor] = None, single_tokens: bool = False):
+    """What enters the recurrence. ``proj`` [tokens, ...] holds q, k, v side by side and the projections of beta and, with one
+    decay per head, of the decay at columns ``b_off`` and ``a_off`` (rows may lie wider apart); ``conv`` float32
+    [taps, channels]; ``z`` (float32 [tokens, >= heads * dim], rows may lie wider apart): the decay's projection per key channel.
+    Returns (act [tokens, channels] in proj's dtype: the convolutions through silu; inv float32 [tokens, 2 kv_heads]: the
+    factors that make query and key heads unit vectors, the queries' with dim ** -0.5; logd float32 [tokens, heads or
+    heads * dim]: the logarithms -exp(a_log) softplus(. + dt_bias) of the decays; beta float32 [tokens, heads]). The
+    convolution's last inputs in ``state`` move on by the step's tokens; ``single_tokens``: every sequence brings one."""
+    _need_cuda(conv, slots, a_log, dt_bias)
+    _check_rows(proj, proj.shape, proj.dtype, "delta_prepare: proj")
+    n, taps, channels = proj.shape[0], conv.shape[0], 2 * kv_heads * dim + heads * v_dim
+    if conv.dtype != torch.float32 or conv.shape[1] != channels:
+        raise KernelError(f"delta_prepare: the convolution's weights are float32 [taps, {channels}]")
+    if state.dtype != torch.float32 or state.shape[1] < (taps - 1) * channels or state.stride(1) != 1:
+        raise KernelError("delta_prepare: the state is float32 [slots, ...] and begins with the convolution's inputs")
+    decays = heads if z is None else heads * dim
+    if a_log.dtype != torch.float32 or a_log.numel() != heads or dt_bias.dtype != torch.float32 or dt_bias.numel() != decays:
+        raise KernelError(f"delta_prepare: a_log is float32 [{heads}] and dt_bias float32 [{decays}]")
+    if z is not None:
+        _check_rows(z, z.shape, torch.float32, "delta_prepare: z")
+        if z.shape[0] != n or z.shape[1] < decays:
+            raise KernelError("delta_prepare: z has a row of heads * dim numbers per token")
+    new = lambda *shape, dtype=torch.float32: torch.empty(shape, dtype=dtype, device=proj.device)
+    act, inv = new(n, channels, dtype=proj.dtype), new(n, 2 * kv_heads)
+    logd, beta = new(n, decays), new(n, heads)
+    _check(lib().ptb_delta_prepare(_dtype_code(proj), _ptr(proj), proj.stride(0), _ptr(conv), _ptr(state), state.stride(0),
+                                   _ptr(slots), ctypes.byref(batch), _ptr(act), _ptr(inv), b_off, a_off, _ptr(z),
+                                   0 if z is None else z.stride(0), _ptr(a_log), _ptr(dt_bias), _ptr(logd), _ptr(beta), heads,
+                                   kv_heads, dim, v_dim, taps, ctypes.c_float(dim ** -0.5), 1 if single_tokens else 0,
+                                   _stream(proj)), "delta_prepare")
+    if not single_tokens and taps > 1:
+        global launches
+        launches += 1       # the kernel that keeps the convolution's last inputs
+    return act, inv, logd, beta
+
+
+def delta_chunks_take(act: torch.Tensor, dim: int, v_dim: int) -> bool:
+    """Does the chunked form on the tensor cores take these sizes? (bfloat16, keys and values of 64 or 128 entries)"""
+    return act.dtype == torch.bfloat16 and bool(lib().ptb_delta_chunks_supports(dim, v_dim))
+
+
+def delta_rule(act: torch.Tensor, inv: torch.Tensor, logd: torch.Tensor, beta: torch.Tensor, state: torch.Tensor,
+               slots: torch.Tensor, batch: StepBatchC, heads: int, kv_heads: int, dim: int, v_dim: int, taps: int,
+               chunks=None) -> torch.Tensor:
+    """Per head S <- diag(exp(l)) S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q over the step's tokens, from and to each
+    sequence's state (after the convolution's inputs, [heads, v_dim, dim]). The first four arguments are what ``delta_prepare``
+    returns. ``chunks``: (chunk_seq, chunk_q0, seq_chunk0, n_chunks) for the chunked form (``delta_chunks_take``), None to walk
+    every sequence token by token. Returns float32 [tokens, heads * v_dim]."""
+    _need_cuda(act, inv, logd, beta, slots)
+    n = act.shape[0]
+    per_head = logd.shape[1] == heads and dim != 1
+    if logd.shape[1] not in (heads, heads * dim) or state.shape[1] < delta_state_floats(heads, kv_heads, dim, v_dim, taps) - 3:
+        raise KernelError("delta_rule: decays are [tokens, heads] or [tokens, heads * dim], the state holds S")
+    out = torch.empty((n, heads * v_dim), dtype=torch.float32, device=act.device)
+    common = (_ptr(state), state.stride(0), _ptr(slots), ctypes.byref(batch))
+    if chunks is None:
+        _check(lib().ptb_delta_walk(_dtype_code(act), _ptr(act), _ptr(inv), _ptr(logd), _ptr(beta), *common, _ptr(out), heads,
+                                    kv_heads, dim, v_dim, taps, 1 if per_head else 0, _stream(act)), "delta_walk")
+        return out
+    chunk_seq, chunk_q0, seq_chunk0, n_chunks = chunks
+    L = lib()
+    L.ptb_delta_chunks_scratch_bytes.restype = ctypes.c_longlong
+    scratch = torch.empty(int(L.ptb_delta_chunks_scratch_bytes(n_chunks, heads, dim, v_dim)), dtype=torch.uint8, device=act.device)
+    _check(L.ptb_delta_chunks(_ptr(act), _ptr(inv), _ptr(logd), _ptr(beta), *common, _ptr(chunk_seq), _ptr(chunk_q0),
+                              _ptr(seq_chunk0), n_chunks, _ptr(scratch), _ptr(out), heads, kv_heads, dim, v_dim, taps,
+                              1 if per_head else 0, _stream(act)), "delta_chunks")
+    global launches
+    launches += 1       # two kernels
+    return out
+
+
+# ------------------------------------------------------------------------------------------------
+# Blocks whose norm comes after the sum; a per-token input
+_POST_NORM = {"branch": 0, "pair": 1, "experts": 2, "add": 3}
+
+
+def _post_norm(kind: str, x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, alpha: float, eps: float, copy_dtype,
+               y2=None, gains=(None, None), gates=None, row_of_pair=None, mult: float = 1.0, eps_branch: float = 0.0):
+    _need_cuda(x, y, y2, gain, gates, row_of_pair, *gains)
+    n, width = x.shape
+    if x.dtype != torch.float32 or gain.dtype != torch.float32 or gain.numel() != width or y.shape[1] != width:
+        raise KernelError("post_norm takes a float32 stream, a float32 gain and branch rows of its width")
+    out = torch.empty_like(x)
+    copy = torch.empty((n, width), dtype=copy_dtype, device=x.device) if copy_dtype not in (None, torch.float32) else None
+    top = 0 if gates is None else gates.shape[1]
+    _check(lib().ptb_post_norm(_POST_NORM[kind], _ptr(x), _dtype_code(y), _ptr(y), _ptr(y2), _ptr(gains[0]), _ptr(gains[1]),
+                               _ptr(gates), _ptr(row_of_pair), top, _ptr(gain), _ptr(out), 0 if copy is None else _dtype_code(copy),
+                               _ptr(copy), n, width, ctypes.c_float(alpha), ctypes.c_float(mult), ctypes.c_float(eps),
+                               ctypes.c_float(eps_branch), _stream(x)), "post_norm")
+    return out, (out if copy is None else copy)
+
+
+def post_norm(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, alpha: float, eps: float, copy_dtype=None):
+    """The float32 stream norm(alpha x + y) * gain (RMS norm) of a branch's result ``y`` (float32 or bfloat16 rows), and the
+    same rounded to ``copy_dtype`` for the sublayers that read it: returns (stream, copy)."""
+    if y.shape != x.shape:
+        raise KernelError("post_norm: the branch's rows have the stream's shape")
+    return _post_norm("branch", x, y, gain, alpha, eps, copy_dtype)
+
+
+def post_norm_pair(x: torch.Tensor, a: torch.Tensor, b: torch.Tensor, gain_a: torch.Tensor, gain_b: torch.Tensor, mult: float,
+                   eps_branch: float, gain: torch.Tensor, alpha: float, eps: float, copy_dtype=None):
+    """``post_norm`` with y = mult (norm(a) gain_a + norm(b) gain_b) of two float32 branches."""
+    if a.dtype != torch.float32 or b.dtype != torch.float32 or a.shape != x.shape or b.shape != x.shape:
+        raise KernelError("post_norm_pair: both branches are float32 rows of the stream's shape")
+    return _post_norm("pair", x, a, gain, alpha, eps, copy_dtype, y2=b, gains=(gain_a, gain_b), mult=mult, eps_branch=eps_branch)
+
+
+def post_norm_experts(x: torch.Tensor, rows: torch.Tensor, row_of_pair: torch.Tensor, gates: torch.Tensor, gain: torch.Tensor,
+                      alpha: float, eps: float, copy_dtype=None):
+    """``post_norm`` with y = the weighed sum of a token's chosen experts' rows (``expert_rows``; no identity experts)."""
+    if rows.dtype != torch.float32 or gates.dtype != torch.float32 or gates.shape[0] != x.shape[0] or row_of_pair.numel() != gates.numel():
+        raise KernelError("post_norm_experts: float32 rows and weights [tokens, top], a row for every choice")
+    return _post_norm("experts", x, rows, gain, alpha, eps, copy_dtype, gates=gates, row_of_pair=row_of_pair)
+
+
+def norm_add(x: torch.Tensor, y: torch.Tensor, gain: torch.Tensor, eps: float, copy_dtype=None):
+    """The float32 stream x + norm(y) * gain (RMS norm) and its copy in ``copy_dtype``: (stream, copy)."""
+    if y.shape != x.shape:
+        raise KernelError("norm_add: the branch's rows have the stream's shape")
+    return _post_norm("add", x, y, gain, 1.0, eps, copy_dtype, eps_branch=eps)
+
+
+def token_gate(z: torch.Tensor, ids: torch.Tensor, table: torch.Tensor, first: int, dim: int, out_width: int,
+               status: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """gelu_tanh(z[t, j]) * table[ids[t], first + j] for j < dim, zeros from there to ``out_width``, in the table's dtype; z float32."""
+    _need_cuda(z, ids, table, status)
+    n = z.shape[0]
+    out = torch.empty((n, out_width), dtype=table.dtype, device=z.device)
+    _check(lib().ptb_token_gate(_dtype_code(z), _ptr(z), z.shape[1], _ptr(ids), _dtype_code(table), _ptr(table), table.shape[0],
+                                table.shape[1], first, _ptr(out), out_width, dim, n, _ptr(status), _stream(z)), "token_gate")
+    return out
+
+
+def round_rows(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """float32 rows in ``dtype`` (bfloat16: rounded; float32: the rows themselves)."""
+    if dtype == torch.float32:
+        return x
+    _need_cuda(x)
+    out = torch.empty(x.shape, dtype=dtype, device=x.device)
+    if x.dtype != torch.float32 or dtype != torch.bfloat16:
+        raise KernelError("round_rows takes float32 rows to bfloat16")
+    _check(lib().ptb_round_rows(_ptr(x), _ptr(out), ctypes.c_longlong(x.numel()), _stream(x)), "round_rows")
     return out

@@ -12,6 +12,8 @@ from ..config.figudra import FigudraConfig
 from .figudra import figudra_spec
 from ..config.vesidra import VesidraConfig
 from .vesidra import vesidra_spec
+from ..config.vabedra import VabedraConfig
+from .vabedra import vabedra_spec
 
 register_architecture(
     "falcon", ("FalconForCausalLM", "RWForCausalLM"), FalconConfig, falcon_spec, name_rules=FALCON_NAME_RULES,
@@ -22,3 +24,4 @@ register_architecture("zalunex", ("Zalunex",), ZalunexConfig, zalunex_spec)
 register_architecture("pogezen", ("Pogezen",), PogezenConfig, pogezen_spec)
 register_architecture("figudra", ("Figudra",), FigudraConfig, figudra_spec)
 register_architecture("vesidra", ("Vesidra",), VesidraConfig, vesidra_spec)
+register_architecture("vabedra", ("Vabedra",), VabedraConfig, vabedra_spec)

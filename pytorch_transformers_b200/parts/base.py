@@ -20,6 +20,8 @@ engine.batch.StepContext of the running step; ``x`` is [tokens, hidden] in the m
                      run: it names the cache entry to read and whether to write it. Optional:
                      ``planner()`` (per-step arrays of its own) and ``runs_beside(ctx)``.
 * ``feed_forward``:  ``forward(x, ctx) -> y``.
+* ``token_input``:   ``forward_stream(x, h, ctx, copy_dtype) -> (x', h')``: what a layer adds to the float32 stream ``x`` (``h``:
+                     its copy in the model dtype) from the tokens' own rows of a table (``ctx.token_table``).
 * ``block``:         ``forward(x, ctx, entry) -> x'`` from its child parts; ``x`` and ``x'`` may be a
                      ``DeferredSum`` (two terms whose sum the next norm forms) or a ``NormedStream`` (a stream with
                      the next block's opening norm already formed); ``resolve`` gives the tensor. ``ctx.next_block``
@@ -35,7 +37,7 @@ from typing import Any, Callable, Dict, List, Optional, Tuple
 
 import torch
 
-FAMILIES = ("norm", "position", "mixer", "feed_forward", "block")
+FAMILIES = ("norm", "position", "mixer", "feed_forward", "token_input", "block")
 _REGISTRY: Dict[str, Dict[str, type]] = {f: {} for f in FAMILIES}
 
 
@@ -123,6 +125,9 @@ class ModelSpec:
     max_positions: int = 0
     # logits <- cap * tanh(logits / cap) after the head (0: none)
     logit_softcap: float = 0.0
+    # a table [vocab, token_table_width] of rows that layers read by token id (parts of the family ``token_input``)
+    token_table_name: Optional[str] = None
+    token_table_width: int = 0
 
     def resolved_schedule(self) -> List[ScheduleEntry]:
         if self.schedule is not None:
@@ -174,7 +179,8 @@ class DeferredSum:
 class NormedStream:
     """A residual stream together with its norm by one norm part (``by``), which the block before computed in the
     kernel that formed the stream because it knew which block runs next (``ctx.next_block``). The block that owns
-    ``by`` uses ``normed``; anybody else takes ``stream``."""
+    ``by`` uses ``normed``; anybody else takes ``stream``. ``by`` None: ``normed`` is the stream itself in the model dtype,
+    for blocks whose sublayers read the stream without a norm."""
     stream: Any
     normed: Any
     by: Any

@@ -191,3 +191,53 @@ class SandwichBlock(Part):
                                    next_dtype=self.build.dtype)
             return NormedStream(x, h, norm)
         return k.post_norm_add(x, y, post.p_weight, post.eps, self.mult)
+
+
+@register_part("block", "post_norm")
+class PostNormBlock(Part):
+    """The norm comes after the sum, and the sublayers read the stream itself:
+
+        x <- norm_mixer(alpha x + mixer(x));      x <- norm_ff(alpha x + ff(x));      then the ``token_input``, if there is one,
+
+    on a float32 residual stream. The stream and its copy in the model dtype, which the sublayers read, come out of one
+    kernel each time; that kernel also norms and sums the two branches of a ``normed_pair`` and weighs and sums the chosen
+    experts' rows of a routed feed-forward. A block without ``feed_forward`` has no ``norm_ff`` either."""
+    graph_safe = True
+
+    def __init__(self, build: BuildContext, spec: PartSpec, alpha: float = 1.0):
+        super().__init__(build, spec)
+        self.alpha = float(alpha)
+        self.mixer, self.norm_mixer = self.children["mixer"], self.children["norm_mixer"]
+        self.feed_forward = self.children.get("feed_forward")
+        self.norm_ff = self.children["norm_ff"] if self.feed_forward is not None else None
+        self.token_input = self.children.get("token_input")
+        for n in (self.norm_mixer, self.norm_ff):
+            if n is not None and (getattr(n, "kind", None) != "rmsnorm" or n.has_bias):
+                raise ValueError("the post-norm block's norms are RMS norms without bias")
+
+    def forward(self, x, ctx, entry):
+        k, dtype = self.build.kernels, self.build.dtype
+        h = x.normed if isinstance(x, NormedStream) and x.by is None else None
+        x = resolve(k, x)
+        if x.dtype != torch.float32:
+            raise ValueError("the post-norm block runs on a float32 residual stream")
+        if h is None:
+            h = k.round_rows(x, dtype)
+        norm = self.norm_mixer
+        if hasattr(self.mixer, "forward_branches"):
+            m = self.mixer
+            left, right = m.forward_branches(h, ctx, entry)
+            x, h = k.post_norm_pair(x, left, right, m.p_left_gain, m.p_right_gain, m.mult, m.eps, norm.p_weight, self.alpha,
+                                    norm.eps, dtype)
+        else:
+            x, h = k.post_norm(x, self.mixer.forward(h, ctx, entry), norm.p_weight, self.alpha, norm.eps, dtype)
+        if self.feed_forward is not None:
+            ff, norm = self.feed_forward, self.norm_ff
+            if getattr(ff, "can_forward_rows", lambda: False)():
+                rows, row_of_pair, weights = ff.forward_rows(h, ctx)
+                x, h = k.post_norm_experts(x, rows, row_of_pair, weights, norm.p_weight, self.alpha, norm.eps, dtype)
+            else:
+                x, h = k.post_norm(x, ff.forward(h, ctx), norm.p_weight, self.alpha, norm.eps, dtype)
+        if self.token_input is not None:
+            x, h = self.token_input.forward_stream(x, h, ctx, dtype)
+        return NormedStream(x, h, None)

@@ -12,6 +12,8 @@ Variants, all by constructor parameters: ``score="sigmoid"`` scores every output
 instead of the softmax; ``correction=False`` has no correction tensor; ``expert="plain"`` experts have no
 gate, ``W_down act(W_up h)`` with ``activation`` by name; ``weight_on="input"`` (plain experts only) multiplies the
 expert's input by the weight instead of its output: the result is the sum of ``expert(weight * h)``.
+``expert="clamped_glu"`` experts clamp their branches: ``W_down (g sigmoid(alpha g) (u + 1))`` with ``g = min(W_gate h, limit)``
+and ``u = clamp(W_up h, -limit, limit)``.
 ``router_bias=True``: the logits are ``W_r h + b``. ``score="softmax_chosen"``: the choice is by the logits (+ correction)
 and the weights are the softmax over the chosen logits alone, times ``scale``.
 ``group_score="top2_sum"`` scores a group by the sum of its two largest choice scores instead of its largest.
@@ -39,7 +41,7 @@ class RoutedExperts(Part):
                  identity: int = 0, groups: int = 1, keep: int = 1, scale: float = 1.0, score: str = "softmax",
                  correction: bool = True, expert: str = "gated_silu", activation: str = "gelu",
                  weight_on: str = "output", group_score: str = "max", normalize: bool = False, shared_gate: bool = False,
-                 router_bias: bool = False):
+                 router_bias: bool = False, limit: float = 0.0, alpha: float = 1.702):
         super().__init__(build, spec)
         if group_score not in ("max", "top2_sum"):
             raise ValueError(f"a group's score is 'max' or 'top2_sum', got {group_score!r}")
@@ -50,13 +52,16 @@ class RoutedExperts(Part):
             raise ValueError("shared_gate needs a shared expert (a child part 'shared')")
         if score not in build.kernels.ROUTE_SCORES:
             raise ValueError(f"router scores are one of {', '.join(build.kernels.ROUTE_SCORES)}, got {score!r}")
-        if expert not in ("gated_silu", "plain") or weight_on not in ("output", "input"):
-            raise ValueError(f"experts are 'gated_silu' or 'plain' and weigh their 'output' or 'input', got {expert!r}, {weight_on!r}")
+        if expert not in ("gated_silu", "clamped_glu", "plain") or weight_on not in ("output", "input"):
+            raise ValueError(f"experts are 'gated_silu', 'clamped_glu' or 'plain' and weigh their 'output' or 'input', got {expert!r}, {weight_on!r}")
         if expert != "plain" and weight_on == "input":
             # the grouped kernels take the weight in the plain expert's first epilogue, or in the sum of outputs
             raise ValueError("gated experts weigh their output")
         if expert == "plain" and (activation not in build.kernels.ACTIVATIONS or identity):
             raise ValueError(f"plain experts take an activation of {', '.join(build.kernels.ACTIVATIONS)} and no identity experts")
+        if (expert == "clamped_glu") != (float(limit) > 0):
+            raise ValueError("experts with a clamped unit have a positive limit, others have none")
+        self.clamp = (float(limit), float(alpha)) if expert == "clamped_glu" else None
         self.weight_on, self.has_router_bias = weight_on, bool(router_bias)
         if normalize and score == "softmax_chosen":
             raise ValueError("the softmax over the chosen logits is normalised already")
@@ -82,7 +87,7 @@ class RoutedExperts(Part):
         if self.has_shared_gate:
             d["shared_gate"] = ParamDecl((1, self.hidden), role="vector")
         for e in range(self.experts):
-            if self.expert == "gated_silu":
+            if self.expert != "plain":
                 d[f"e{e}.gate"] = ParamDecl((self.inner, self.hidden))
             d[f"e{e}.up"] = ParamDecl((self.inner, self.hidden))
             d[f"e{e}.down"] = ParamDecl((self.hidden, self.inner))
@@ -107,6 +112,19 @@ class RoutedExperts(Part):
             down[e] = t.pop(f"e{e}.down")
         self.p_gate_up, self.p_down = gate_up, down
 
+    def can_forward_rows(self) -> bool:
+        """Experts alone, weighed on their output: their rows can be summed by the kernel that norms the sum."""
+        return self.shared is None and self.identity == 0 and self.weight_on == "output"
+
+    def forward_rows(self, x, ctx):
+        """The chosen experts' rows before they are summed: (float32 rows, row of every choice, weights [tokens, top])."""
+        k = self.build.kernels
+        ids, weights = k.route(x, self.p_router, self.p_correction, self.groups, self.keep, self.top, self.scale, self.score,
+                               group_top=2 if self.group_score == "top2_sum" else 1, normalize=self.normalize, bias=self.p_router_b)
+        rows, row_of_pair = k.expert_rows(x, ids, self.p_gate_up, self.p_down,
+                                          plain_act=self.activation if self.expert == "plain" else None, clamp=self.clamp)
+        return rows, row_of_pair, weights
+
     def forward(self, x, ctx, add=None):
         k = self.build.kernels
         if callable(add):
@@ -122,4 +140,4 @@ class RoutedExperts(Part):
                 shared_gate = routed[2][:, self.experts + self.identity:]
         return k.routed_experts(x, ids, weights, self.p_gate_up, self.p_down, base=add,
                                 plain_act=self.activation if self.expert == "plain" else None, shared=shared,
-                                shared_gate=shared_gate, weigh_output=self.weight_on == "output")
+                                shared_gate=shared_gate, weigh_output=self.weight_on == "output", clamp=self.clamp)

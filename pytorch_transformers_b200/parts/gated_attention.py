@@ -14,7 +14,8 @@
   1 + coef ln(floor((p + 1) / every) + 1);
 * a norm with gains that comes before the rotation (``norm_first``);
 * values of a size of their own (``vdim``);
-* biases on the four projections (``bias``), added in float32 where queries, keys and values are laid out;
+* biases on the four projections (``bias``; ``out_bias=False``: not on the output's), added in float32 where queries, keys and
+  values are laid out;
 * a rotation of queries and keys from a ``position`` child, applied before the norm of queries and keys, and a
   norm without gains (``qk_gain=False``: plain division by the root mean square);
 * first positions that stay visible left of the window (``keep_first``): i sees j if j <= i and
@@ -48,7 +49,7 @@ class SinkAttention(Part):
                  scale: float, window: int = 0, eps: float = 1e-6, qk_norm: bool = True, sink: bool = True,
                  gate: bool = True, bias: bool = False, qk_gain: bool = True, keep_first: int = 0, talk: bool = False,
                  value_mix: str = "none", value_mix_key: str = "values", softcap: float = 0.0, q_temp=None,
-                 gate_wide: bool = False, sink_value=None, norm_first: bool = False):
+                 gate_wide: bool = False, sink_value=None, norm_first: bool = False, out_bias: bool = True):
         super().__init__(build, spec)
         if heads % kv_heads:
             raise ValueError(f"heads ({heads}) must be a multiple of kv_heads ({kv_heads})")
@@ -78,6 +79,7 @@ class SinkAttention(Part):
             raise ValueError("mixed softmax weights go with neither a sink nor a soft cap")
         if self.norm_first and not (self.qk_norm and self.qk_gain):
             raise ValueError("norm_first is the norm with gains before the rotation (qk_norm and qk_gain)")
+        self.has_out_bias = self.has_bias and bool(out_bias)
         self.gate_cols = (self.heads * self.vdim if self.gate_wide else self.heads) if self.has_gate else 0
         self.position = self.children.get("position")
         # the second path: rotation, biases, kept first positions, mixed weights or mixed values
@@ -100,7 +102,9 @@ class SinkAttention(Part):
             decls["g"] = ParamDecl((self.gate_cols, self.hidden))
         if self.has_bias:
             decls.update({"q_b": ParamDecl((H * d,), role="vector", std=0.5), "k_b": ParamDecl((G * d,), role="vector", std=0.5),
-                          "v_b": ParamDecl((G * vd,), role="vector", std=0.5), "o_b": ParamDecl((self.hidden,), role="vector")})
+                          "v_b": ParamDecl((G * vd,), role="vector", std=0.5)})
+            if self.has_out_bias:
+                decls["o_b"] = ParamDecl((self.hidden,), role="vector")
             if self.has_gate:
                 decls["g_b"] = ParamDecl((self.gate_cols,), role="vector")
         if self.talk:
@@ -118,7 +122,7 @@ class SinkAttention(Part):
             self.p_sink = torch.full((self.heads,), self.sink_value, dtype=torch.float32, device=t["q"].device)
         if self.has_bias:
             self.p_in_b = torch.cat([t["q_b"], t["k_b"], t["v_b"]] + ([t["g_b"]] if self.has_gate else [])).contiguous()
-            self.p_o_b = t["o_b"]
+            self.p_o_b = t.get("o_b")
         self.p_talk, self.p_vmix = t.get("talk"), t.get("vmix")
 
     # ---- the projected protocol (parts/pair.py)

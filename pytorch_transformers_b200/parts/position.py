@@ -33,7 +33,7 @@ class NoPosition(Part):
 @register_part("position", "rotary")
 class RotaryPosition(NoPosition):
     def __init__(self, build: BuildContext, spec: PartSpec, head_dim: int, theta: float, factor: float = 1.0,
-                 rotary_dim: int = 0, interleaved: bool = False, yarn: dict = None):
+                 rotary_dim: int = 0, interleaved: bool = False, yarn: dict = None, bands: dict = None):
         super().__init__(build, spec)
         # which dims make a rotated pair: (i, i + dim / 2), the reference's rotate_half, or (2 i, 2 i + 1)
         self.interleaved = bool(interleaved)
@@ -47,9 +47,12 @@ class RotaryPosition(NoPosition):
         self.table_scale = 1.0
         if yarn:
             inv_freq, self.table_scale = yarn_frequencies(dim, float(theta), **yarn)
+        if bands:
+            inv_freq = banded_frequencies(dim, float(theta), **bands)
         self.inv_freq = inv_freq.to(torch.float32).to(build.device)
         # layers whose rotation has the same constants share one table of angles per step
-        self.rotation_key = ("rotary", dim, float(theta), float(factor), tuple(sorted((yarn or {}).items())))
+        self.rotation_key = ("rotary", dim, float(theta), float(factor), tuple(sorted((yarn or {}).items())),
+                             tuple(sorted((bands or {}).items())))
 
     def rotation(self):
         return self.inv_freq
@@ -72,6 +75,17 @@ def yarn_frequencies(dims: int, base: float, factor: float, original: float, fas
     hi = min(math.ceil(index_of(slow)), dims - 1)
     ramp = torch.clamp((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
     return f / float(factor) * ramp + f * (1.0 - ramp), 0.1 * math.log(float(factor)) + 1.0
+
+
+def banded_frequencies(dims: int, base: float, factor: float, low: float, high: float, original: float) -> torch.Tensor:
+    """Frequencies scaled by their wavelength l = 2 pi / f (the scaling of Llama 3.1): kept where l < original / high, divided
+    by ``factor`` where l > original / low, and in between (1 - s) f / factor + s f with
+    s = (original / l - low) / (high - low). Computed in float64; [dims / 2]."""
+    f = float(base) ** (-2.0 * torch.arange(dims // 2, dtype=torch.float64) / dims)
+    turns = float(original) * f / (2.0 * math.pi)          # original / l
+    s = (turns - float(low)) / (float(high) - float(low))
+    mixed = (1.0 - s) * f / float(factor) + s * f
+    return torch.where(turns > float(high), f, torch.where(turns < float(low), f / float(factor), mixed))
 
 
 def alibi_slopes(heads: int) -> torch.Tensor:
