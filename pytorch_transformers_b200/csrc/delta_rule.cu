@@ -16,7 +16,7 @@
 
 namespace {
 
-constexpr int MAX_TAPS = 8;
+constexpr int MAX_TAPS = 64;
 constexpr int PREP_WARPS = 8;
 constexpr float UNIT_EPS = 1e-6f;     // inside the root of the unit vectors' norm
 

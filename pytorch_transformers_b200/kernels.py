@@ -1504,7 +1504,7 @@ def gla(proj: torch.Tensor, log_decay: torch.Tensor, state: torch.Tensor, slots:
 # ------------------------------------------------------------------------------------------------
 # The gated delta rule
 DELTA_MAX_DIM = 256   # ptb_delta_max_dim()
-DELTA_MAX_TAPS = 8    # ptb_delta_max_taps()
+DELTA_MAX_TAPS = 64   # ptb_delta_max_taps()
 DELTA_CHUNK = 64      # ptb_delta_chunk_tokens()
 
 
