@@ -572,7 +572,9 @@ class KernelTimes:
              "latent_unfolded_attention",
              "latent_expand", "block_linear", "rglru_conv", "rglru_scan", "rglru_scan_chunks", "route", "routed_experts", "scale_",
              "embed_sum", "post_norm_add", "qk_norm_store", "linear_attention", "norm_gate", "glu_clamp", "softcap_",
-             "dyt", "mlstm", "head_norm_gate", "rope_norm_store", "talk_mix", "embed_rows", "gla", "gla_decay_", "glu_act")
+             "dyt", "mlstm", "head_norm_gate", "rope_norm_store", "talk_mix", "embed_rows", "gla", "gla_decay_", "glu_act",
+             "delta_prepare", "delta_rule", "expert_rows", "post_norm", "post_norm_pair", "post_norm_experts", "norm_add", "token_gate",
+             "round_rows")
 
     def __init__(self, kernels):
         self.k, self.records, self.saved = kernels, [], {}
@@ -1167,7 +1169,116 @@ def run_vesidra(args):
     return 0
 
 
+# ---- Vabedra beside Figudra at equal size (`--only vabedra [--size s|m]`) ----
+# Sizes that resemble a served model's layers: the width; four layers that take turns, an attention beside a delta rule (16
+# or 32 heads of 128 on a quarter as many K/V heads with biases, normed and partly rotated queries and keys with frequencies
+# scaled by wavelength, capped scores, a window of 1,024 that keeps the first 4 tokens and one added to the denominator; as
+# many delta heads of 128 x 128 with a decay per key channel, decay and gate through ranks of 64, filters of 4 taps) and a
+# delta rule alone (as many heads with one decay a head, two of them on a query/key head), each over 64 experts of 1,408 with
+# clamped units of which a token uses 6, and a token input of 64 columns. Figudra beside it is `--only figudra`'s model of
+# the same width, heads and experts: the library's other design with a state of 128 x 128 a head, a decay per key channel, a
+# windowed attention that keeps the first tokens and gated experts.
+def vabedra_config(size):
+    z = PAFEVIK_SIZES[size]
+    w, heads = z["width"], z["heads"]
+    left = {"heads": heads, "kv_heads": heads // 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "softcap": 30.0,
+            "mask": {"size": 1024, "keep_first": 4},
+            "rot": {"base": 10000.0, "dims": 64, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}}
+    right = {"heads": heads, "kv_heads": heads, "dim": 128, "vdim": 128, "conv": 4, "rank": 64}
+    alone = {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": 1408, "limit": 7.0}, "router": {"experts": 64, "top": 6}}
+    pair = {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": moe}
+    return {"architecture": "Vabedra", "vocab": 32000, "width": w, "norm": {"eps": 1e-6}, "postln_alpha": 2.0,
+            "embedding": {"scale": w ** 0.5}, "token_side": {"dim": 64},
+            "layers": [pair, {"type": "delta", "mixer": alone, "mlp": moe}] * 2}
+
+
+def run_vabedra(args):
+    import torch
+
+    import pytorch_transformers_b200 as ptb
+
+    torch.cuda.set_device(0)
+    pk = peaks()
+    gen = torch.Generator().manual_seed(0)
+    tokens, batch, context = args.prefill_tokens, args.batch, args.context
+    raw, fig = vabedra_config(args.size), figudra_config(args.size)
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
+    left, right, w = raw["layers"][0]["mixer"]["left"], raw["layers"][0]["mixer"]["right"], raw["width"]
+    result = {"only": "vabedra", "size": args.size, "prefill_tokens": tokens, "batch": batch, "context": context,
+              "config": {"width": w, "layers": len(raw["layers"]), "heads": left["heads"]}}
+    for name, cfg in (("vabedra", ptb.VabedraConfig.from_dict(raw)), ("figudra", ptb.FigudraConfig.from_dict(fig))):
+        model = ptb.AutoModelForCausalLM.from_config(cfg, seed=0, dtype="bfloat16")
+        result[name] = measure_prefill_and_decode(model, args, gen, flush)
+        del model
+        torch.cuda.empty_cache()
+    V, F = result["vabedra"]["prefill_kernels_ms"], result["figudra"]["prefill_kernels_ms"]
+    VD, FD = result["vabedra"]["decode_kernels_ms"], result["figudra"]["decode_kernels_ms"]
+
+    def per_call(table, key):
+        return table[key]["ms"] / table[key]["calls"] if key in table else None
+
+    roof = {}
+
+    def rate(name, t, flops=None, moved=None):
+        """Achieved rates of a call of t ms against the measured peaks: operations, bytes or both."""
+        if not t:
+            return
+        if flops is not None:
+            roof[f"{name}_TFLOPs"] = round(flops / t / 1e9, 1)
+            roof[f"{name}_frac_of_burst"] = round(flops / t / 1e9 / pk["bf16_tflops"], 4)
+        if moved is not None:
+            roof[f"{name}_GBps"] = round(moved / t / 1e6, 1)
+            roof[f"{name}_frac_of_hbm"] = round(moved / t / 1e6 / pk["hbm_gbs"], 4)
+
+    H, G, d, vd = left["heads"], left["kv_heads"], left["dim"], left["vdim"]
+    keep, size = left["mask"]["keep_first"], left["mask"]["size"]
+    seen = sum(min(t + 1, size) + max(0, min(keep, t + 1 - size)) for t in range(tokens))
+    full = tokens * (tokens + 1) // 2
+    rate("attention_prefill", per_call(V, "attention_mma"), flops=H * seen * 2 * (d + vd))
+    if "attention_mma" in F:    # one windowed and one full layer share the table's row
+        rate("figudra_attention_prefill", F["attention_mma"]["ms"], flops=H * (seen + full) * 2 * (d + vd))
+    # the delta rule: queries, keys and values in, decays in (per channel in two layers, per head in two), float32 rows out;
+    # what it needs a token and head: the read at the key, the write and the read at the query, 3 dim vdim multiply-adds
+    lh, ld, lv = right["heads"], right["dim"], right["vdim"]
+    io = tokens * lh * (2 * (2 * ld + lv) + (4 * ld + 4) / 2 + 4 * lv)
+    rate("delta_rule_prefill", per_call(V, "delta_rule"), flops=lh * tokens * 2 * 3 * ld * lv, moved=io)
+    rate("figudra_gla_prefill", per_call(F, "gla"), flops=lh * tokens * 2 * 3 * ld * lv, moved=tokens * lh * (2 * (2 * ld + lv) + 4 * ld + 4 * lv))
+    # half of the calls form decays per channel (float32 in and out); half have two heads on a query/key head
+    rate("delta_prepare_prefill", per_call(V, "delta_prepare"), moved=tokens * lh * (4 * (ld + ld / 2 + lv) + 8 * ld / 2))
+    rate("figudra_gla_decay_prefill", per_call(F, "gla_decay_"), moved=tokens * lh * ld * 8)
+    pairs = tokens * 6
+    rate("expert_rows_prefill", per_call(V, "expert_rows"), flops=pairs * 3 * 2 * w * 1408)
+    rate("figudra_expert_rows_prefill", per_call(F, "expert_rows"), flops=pairs * 3 * 2 * w * 1408)
+    rate("post_norm_pair_prefill", per_call(V, "post_norm_pair"), moved=tokens * w * (4 * 4 + 2))
+    rate("post_norm_prefill", per_call(V, "post_norm"), moved=tokens * w * (3 * 4 + 2))
+    rate("post_norm_experts_prefill", per_call(V, "post_norm_experts"), moved=tokens * w * (2 * 4 + 6 * 4 + 2))
+    rate("norm_add_prefill", per_call(V, "norm_add"), moved=tokens * w * (3 * 4 + 2))
+    rate("figudra_norm_stream_prefill", per_call(F, "norm_stream"), moved=tokens * w * (4 + 4 + 4 + 2))
+    rate("head_norm_gate_prefill", per_call(V, "head_norm_gate"), moved=tokens * lh * lv * (4 + 3 + 2))      # half of the gates float32
+    rate("figudra_head_norm_gate_prefill", per_call(F, "head_norm_gate"), moved=tokens * lh * lv * (4 + 2 + 2))
+    rows = tokens * ((H + G) * d + G * vd) * 4
+    rate("rope_norm_store_prefill", per_call(V, "rope_norm_store"), moved=rows)
+    rate("figudra_rope_norm_store_prefill", per_call(F, "rope_norm_store"), moved=rows)
+    if "matmul_nt" in V:        # all library products of the prompt
+        n_att = 2 * ((H + G) * d + G * vd + H * vd)
+        n_pair = 2 * (2 * lh * ld + 2 * lh * lv + lh + 128)
+        n_alone = 2 * (lh * ld + 3 * lh * lv + 2 * lh)
+        flops = 2 * tokens * (w * (n_att + n_pair + n_alone) + 2 * 128 * lh * (ld + lv) + 4 * 2 * 64 * w)
+        rate("library_products", V["matmul_nt"]["ms"], flops=flops)
+    # single tokens, launched one by one: event pairs around small kernels hold the launch too
+    state = batch * lh * ld * lv * 8
+    rate("delta_rule_decode", per_call(VD, "delta_rule"), moved=state)
+    rate("figudra_gla_decode", per_call(FD, "gla"), moved=state)
+    result["roofline"] = roof
+    result["peaks"] = pk
+    print(json.dumps(result))
+    return 0
+
+
 def run_ours(args):
+    if args.only == "vabedra":
+        return run_vabedra(args)
     if args.only == "vesidra":
         return run_vesidra(args)
     if args.only == "figudra":
@@ -1453,10 +1564,10 @@ def main():
     ap.add_argument("--layers", type=int, default=0, help="fewer layers than the configuration's (0: all)")
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--only", default="", choices=["", "decode", "prefill", "sample", "decode-attention", "prefill-attention", "config", "linear",
-                             "fill", "mma-cadence", "pafevik", "zalunex", "pogezen", "figudra", "vesidra"],
+                             "fill", "mma-cadence", "pafevik", "zalunex", "pogezen", "figudra", "vesidra", "vabedra"],
                     help="run one section only and print its numbers (for profilers)")
     ap.add_argument("--shape", default="7b", choices=sorted(SHAPES), help="model shape for --only decode / prefill")
-    ap.add_argument("--size", default="s", choices=sorted(PAFEVIK_SIZES), help="layer sizes for --only pafevik, --only zalunex, --only pogezen, --only figudra and --only vesidra")
+    ap.add_argument("--size", default="s", choices=sorted(PAFEVIK_SIZES), help="layer sizes for --only pafevik, --only zalunex, --only pogezen, --only figudra, --only vesidra and --only vabedra")
     ap.add_argument("--prefill-tokens", type=int, default=PREFILL_TOKENS, help="prompt length for --only prefill")
     ap.add_argument("--context", type=int, default=CONTEXT, help="cached tokens per sequence for --only decode")
     ap.add_argument("--past", type=int, default=0, help="cached tokens before the prompt for --only prefill-attention")
