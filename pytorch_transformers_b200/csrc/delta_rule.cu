@@ -18,6 +18,8 @@ namespace {
 
 constexpr int MAX_TAPS = 64;
 constexpr int PREP_WARPS = 8;
+constexpr int PREP_RUN = 8;           // tokens of a warp in steps of many tokens
+constexpr int FAST_TAPS = 4;          // the filter length whose inputs are held in registers
 constexpr float UNIT_EPS = 1e-6f;     // inside the root of the unit vectors' norm
 
 __device__ __forceinline__ float silu_of(float v) { return v / (1.f + expf(-v)); }
@@ -65,7 +67,7 @@ struct DeltaSizes {
   __host__ __device__ int channels() const { return 2 * kv_heads * dim + heads * v_dim; }
 };
 
-// A warp per (run of RT tokens, unit). Units: the 2 kv_heads query and key heads (convolution, silu, inverse norm), the
+// A warp per (run of RUN tokens, unit). Units: the 2 kv_heads query and key heads (convolution, silu, inverse norm), the
 // values in stretches of 128 channels (convolution, silu), the decays' logarithms per channel in stretches of 128
 // (DECAY_CHANNEL), and one unit with beta and the decays' logarithms per head.
 //   proj row t: [q | k | v] then, at b_off and a_off, the projections of beta and of the decay per head; z (float32 rows
@@ -73,19 +75,89 @@ struct DeltaSizes {
 //   act [tokens][channels] (T): the activated convolutions, rounded to T; inv [tokens][2 kv_heads]: what a query and a key
 //   head is multiplied by to be a unit vector (queries: also dim^-1/2); logd [tokens][heads * dim or heads]; beta [tokens][heads].
 // With `single` (one new token a sequence) the convolution's kept inputs are moved on here, each by the thread that read it.
-template <typename T, int V>
+//
+// RUN > 1 (steps of many tokens): a warp's RUN neighbouring tokens of one sequence under a filter of FAST_TAPS taps have all
+// their inputs loaded before the first is used, each once; runs that span sequences, other taps and wide heads go token by
+// token. The sums are formed in the same order either way.
+template <typename T, int V, int RUN>
 __global__ void __launch_bounds__(32 * PREP_WARPS)
 delta_prepare_kernel(const T* __restrict__ proj, int stride, const float* __restrict__ conv_w, float* __restrict__ state,
                      int state_stride, const int* __restrict__ slots, StepBatch sb, T* __restrict__ act,
                      float* __restrict__ inv, int b_off, int a_off, const float* __restrict__ z, int z_stride,
                      const float* __restrict__ a_log, const float* __restrict__ dt_bias, float* __restrict__ logd,
-                     float* __restrict__ beta, DeltaSizes sz, int run, int single, float q_scale) {
+                     float* __restrict__ beta, DeltaSizes sz, int single, float q_scale) {
   const int warp = threadIdx.x / 32, lane = threadIdx.x % 32;
   const int C = sz.channels(), qk = sz.qk(), hv = sz.heads * sz.v_dim, hd = sz.heads * sz.dim, keep = sz.taps - 1;
   const int n_heads = 2 * sz.kv_heads, n_v = (hv + 127) / 128, n_d = z ? (hd + 127) / 128 : 0;
   const int unit = blockIdx.y * PREP_WARPS + warp;
   if (unit > n_heads + n_v + n_d) return;
-  const int t0 = blockIdx.x * run, t1 = min(t0 + run, sb.n_tokens);
+  const int t0 = blockIdx.x * RUN, t1 = min(t0 + RUN, sb.n_tokens);
+  if (z != nullptr && unit >= n_heads + n_v && unit < n_heads + n_v + n_d) {
+    const int c0 = (unit - n_heads - n_v) * 128;
+    if (V == 4 && (z_stride & 3) == 0) {       // four channels of one head a lane (the host checks: dim a multiple of 4)
+      const int c = c0 + lane * 4;
+      if (c >= hd) return;
+      const float a = -expf(a_log[c / sz.dim]);
+      const Vals<V> bias = load_vals<V>(dt_bias + c);
+#pragma unroll 4
+      for (int t = t0; t < t1; ++t) {
+        Vals<V> x = load_vals<V>(z + size_t(t) * z_stride + c);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x.f[e] = a * softplus_of(x.f[e] + bias.f[e]);
+        store_vals<V>(logd + size_t(t) * hd + c, x);
+      }
+      return;
+    }
+    for (int u = 0; u < 4; ++u) {
+      const int c = c0 + u * 32 + lane;
+      if (c >= hd) return;
+      const float a = -expf(a_log[c / sz.dim]);
+      for (int t = t0; t < t1; ++t) logd[size_t(t) * hd + c] = a * softplus_of(z[size_t(t) * z_stride + c] + dt_bias[c]);
+    }
+    return;
+  }
+  if constexpr (RUN > 1) {
+    constexpr int KEEP = FAST_TAPS - 1;
+    const bool norm = unit < n_heads;
+    const int c0 = norm ? unit * sz.dim : 2 * qk + (unit - n_heads) * 128, n = norm ? sz.dim : min(128, C - c0);
+    const int seq = sb.tok_seq[t0];
+    if (unit < n_heads + n_v && sz.taps == FAST_TAPS && n <= 32 * V && t1 == t0 + RUN && sb.tok_seq[t1 - 1] == seq) {
+      const int i0 = t0 - sb.seq_start[seq], c = c0 + lane * V;
+      const bool on = lane * V < n;
+      Vals<V> x[KEEP + RUN], w[FAST_TAPS];
+      if (on) {
+        const float* st = state + size_t(slots[seq]) * state_stride + c;
+#pragma unroll
+        for (int r = 0; r < KEEP + RUN; ++r) {
+          const int li = i0 + r - KEEP;
+          x[r] = li >= 0 ? load_vals<V>(proj + size_t(t0 + r - KEEP) * stride + c) : load_vals<V>(st + size_t(KEEP + li) * C);
+        }
+#pragma unroll
+        for (int tap = 0; tap < FAST_TAPS; ++tap) w[tap] = load_vals<V>(conv_w + size_t(tap) * C + c);
+      }
+#pragma unroll
+      for (int r = 0; r < RUN; ++r) {
+        float ss = 0.f;
+        if (on) {
+          Vals<V> y;
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            float v = 0.f;
+#pragma unroll
+            for (int tap = 0; tap < FAST_TAPS; ++tap) v = fmaf(w[tap].f[e], x[r + tap].f[e], v);
+            y.f[e] = to_f(from_f<T>(silu_of(v)));
+            ss = fmaf(y.f[e], y.f[e], ss);
+          }
+          store_vals<V>(act + size_t(t0 + r) * C + c, y);
+        }
+        if (norm) {
+          const float q = 1.0f / sqrtf(warp_sum(ss) + UNIT_EPS);
+          if (lane == 0) inv[size_t(t0 + r) * n_heads + unit] = unit < sz.kv_heads ? q * q_scale : q;
+        }
+      }
+      return;
+    }
+  }
   for (int t = t0; t < t1; ++t) {
     if (unit < n_heads + n_v) {
       const int seq = sb.tok_seq[t], i = t - sb.seq_start[seq];
@@ -122,14 +194,6 @@ delta_prepare_kernel(const T* __restrict__ proj, int stride, const float* __rest
       if (norm) {
         const float r = 1.0f / sqrtf(warp_sum(ss) + UNIT_EPS);
         if (lane == 0) inv[size_t(t) * n_heads + unit] = unit < sz.kv_heads ? r * q_scale : r;
-      }
-    } else if (unit < n_heads + n_v + n_d) {
-      const int c0 = (unit - n_heads - n_v) * 128;
-#pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int c = c0 + u * 32 + lane;
-        if (c < hd)
-          logd[size_t(t) * hd + c] = -expf(a_log[c / sz.dim]) * softplus_of(z[size_t(t) * z_stride + c] + dt_bias[c]);
       }
     } else {
       for (int h = lane; h < sz.heads; h += 32) {
@@ -309,24 +373,28 @@ PTB_API int ptb_delta_prepare(int dtype, const void* proj, int stride, const flo
     return PTB_ERR_SIZE;
   if (dtype != PTB_F32 && dtype != PTB_BF16) return PTB_ERR_DTYPE;
   const int hv = heads * v_dim, units = 2 * kv_heads + (hv + 127) / 128 + (z ? (heads * dim + 127) / 128 : 0) + 1;
-  const int run = sb->n_tokens >= 8 * sm_count() ? 4 : 1;       // tokens of a warp
+  const int run = sb->n_tokens >= 4 * sm_count() ? PREP_RUN : 1;
   const dim3 grid((sb->n_tokens + run - 1) / run, (units + PREP_WARPS - 1) / PREP_WARPS);
   if (grid.y > 65535) return PTB_ERR_SIZE;
   const size_t word = dtype == PTB_F32 ? 16 : 8;
   const bool vec = dim % 4 == 0 && hv % 4 == 0 && stride % 4 == 0 && state_stride % 4 == 0 &&
                    reinterpret_cast<uintptr_t>(proj) % word == 0 && reinterpret_cast<uintptr_t>(act) % word == 0 &&
-                   aligned16(conv_w) && (taps == 1 || aligned16(state));
-#define PTB_PREP(TT, VV)                                                                                                       \
-  delta_prepare_kernel<TT, VV><<<grid, 32 * PREP_WARPS, 0, stream>>>((const TT*)proj, stride, conv_w, state, state_stride, slots, \
-                                                                     *sb, (TT*)act, inv, b_off, a_off, z, z_stride, a_log,       \
-                                                                     dt_bias, logd, beta, sz, run, single, q_scale)
-  if (dtype == PTB_F32) {
-    if (vec) PTB_PREP(float, 4);
-    else PTB_PREP(float, 1);
-  } else {
-    if (vec) PTB_PREP(__nv_bfloat16, 4);
-    else PTB_PREP(__nv_bfloat16, 1);
-  }
+                   aligned16(conv_w) && (taps == 1 || aligned16(state)) &&
+                   (z == nullptr || (aligned16(z) && aligned16(dt_bias)));
+#define PTB_PREP2(TT, VV, RR)                                                                                                  \
+  delta_prepare_kernel<TT, VV, RR><<<grid, 32 * PREP_WARPS, 0, stream>>>((const TT*)proj, stride, conv_w, state, state_stride, \
+                                                                         slots, *sb, (TT*)act, inv, b_off, a_off, z, z_stride,  \
+                                                                         a_log, dt_bias, logd, beta, sz, single, q_scale)
+#define PTB_PREP(TT)                                        \
+  do {                                                      \
+    if (vec && run > 1) PTB_PREP2(TT, 4, PREP_RUN);         \
+    else if (vec) PTB_PREP2(TT, 4, 1);                      \
+    else if (run > 1) PTB_PREP2(TT, 1, PREP_RUN);           \
+    else PTB_PREP2(TT, 1, 1);                               \
+  } while (0)
+  if (dtype == PTB_F32) PTB_PREP(float);
+  else PTB_PREP(__nv_bfloat16);
+#undef PTB_PREP2
 #undef PTB_PREP
   if (launch_status() != PTB_OK) return PTB_ERR_LAUNCH;
   if (single || taps == 1) return PTB_OK;

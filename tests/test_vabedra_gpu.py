@@ -185,6 +185,25 @@ def test_what_enters_the_recurrence(m, channel, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("m,channel", [(vm.delta(4, 2, 24, 20, 4), False), (vm.delta(2, 2, 64, 40, 4, rank=5), True),
+                                       (vm.delta(2, 1, 9, 6, 4, rank=3), True), (vm.delta(2, 1, 32, 32, 3), False),
+                                       (vm.delta(1, 1, 144, 16, 4), False)], ids=lambda v: str(v) if isinstance(v, bool) else f"{v['dim']}x{v['conv']}")
+def test_steps_of_many_tokens_form_the_same_inputs(m, channel, dtype):
+    """Hundreds of tokens of several sequences in one step, after a first portion of a few tokens each: runs of tokens whose
+    inputs reach into the portion before, that span two sequences and that end with the step."""
+    width, lengths, heads = 48, [333, 9, 7, 420, 2], [3, 1, 2, 5, 1]
+    mixer, w = delta_part(m, width, channel, dtype, seed=5)
+    g = torch.Generator().manual_seed(6)
+    xs = [bf16_exact(torch.randn(n, width, generator=g)).float() for n in lengths]
+    cache = mixer.cache(64 * 20, max_slots=5)
+    slots = [cache.open() for _ in xs]
+    first = mixer.step(cache, slots, [x[:h] for x, h in zip(xs, heads)])
+    second = mixer.step(cache, slots, [x[h:] for x, h in zip(xs, heads)])
+    for x, a, b in zip(xs, first, second):
+        close(torch.cat([a, b]), plain.delta_mixer(x.double(), w, m, 1e-5), dtype, f"{len(x)} tokens", f32=4e-5)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("m,channel", DELTAS, ids=[_did(v) for v in DELTAS])
 def test_delta_rule_whole_in_portions_in_chunks_and_token_by_token(m, channel, dtype):
     width = 48
